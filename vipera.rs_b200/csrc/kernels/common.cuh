@@ -37,7 +37,14 @@ template <>
 __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
 // Activations of a gated unit's gate, or of a unit without a gate.
-enum ViperaActivation { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2 };
+enum ViperaActivation { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2, ACT_CLAMPED = 3 };
+
+// ACT_CLAMPED, a gated unit whose two halves are bounded: g = min(gate, limit), u = up held within
+// +-limit; g * sigmoid(slope * g) * (u + 1).
+__device__ __forceinline__ float clamped_unit(float gate, float up, float limit, float slope) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+}
 
 __device__ __forceinline__ float gate_activation(float z, int activation) {
   if (activation == ACT_GELU_TANH)

@@ -73,7 +73,7 @@ struct GemmParams {
   int epilogue;
   int out_dtype;
   const float* bias;  // [N] or null; counts in every ending (in the gated unit: interleaved like the rows)
-  int activation;     // of the gated unit: ACT_SILU or ACT_GELU_TANH
+  int activation;     // of the gated unit: ACT_SILU, ACT_GELU_TANH or (grouped) ACT_CLAMPED
   void* out;
   float* resid;
   int tma_ending;    // 1: the ending goes through shared memory and TMA stores (map_out)
@@ -98,6 +98,8 @@ struct GemmParams {
   // The table is written by a kernel ahead of this one, so no weight tile is fetched before it.
   const int* tile_group;     // [tiles_x] or null
   int group_stride;          // rows of W from one matrix to the next (N)
+  const float* unit_limit;   // grouped, ACT_CLAMPED: [groups] the bound of each group's gated unit
+  float unit_slope;          // and the slope inside its sigmoid
 };
 
 // ---------------------------------------------------------------------------------------
@@ -283,9 +285,17 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
 }
 // up * silu(gate); the quotient with the hardware's reciprocal (the result is rounded to
 // bfloat16 by every caller on the tensor-core path, which hides the last bits)
+__device__ __forceinline__ float silu_mul_slope(float gate, float up, float slope) {
+  return up * __fdividef(gate, 1.0f + __expf(-slope * gate));
+}
 __device__ __forceinline__ float silu_mul(float gate, float up) { return up * __fdividef(gate, 1.0f + __expf(-gate)); }
-// The gated unit: up * act(gate).
-__device__ __forceinline__ float glu_mul(float gate, float up, int activation) {
+// The gated unit: up * act(gate), or the bounded unit (`limit` and `slope` count there only), whose
+// result is rounded to bfloat16 as well.
+__device__ __forceinline__ float glu_mul(float gate, float up, int activation, float limit = 0.0f, float slope = 0.0f) {
+  if (activation == ACT_CLAMPED) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return silu_mul_slope(g, u + 1.0f, slope);
+  }
   if (activation == ACT_GELU_TANH) return up * gate_activation(gate, ACT_GELU_TANH);
   return silu_mul(gate, up);
 }
@@ -318,6 +328,11 @@ struct TileConfig {
 // SWAP = true : accumulator rows are features, columns are tokens.
 // EXT: the ending knows a bias outside the plain store and the gated unit's other activation; the
 // instances without it are the kernels as they were before those options existed.
+// The bound of the gated units of tile tx (whose group a kernel ahead wrote); 0 where no unit has one.
+__device__ __forceinline__ float unit_limit_of(const GemmParams& p, int tx) {
+  return p.activation == ACT_CLAMPED ? p.unit_limit[p.tile_group[tx]] : 0.0f;
+}
+
 template <int BN, bool SWAP, bool EXT = false>
 __device__ __forceinline__ void finish_chunk(const GemmParams& p, const float* v, int width, int row, int col0) {
   // `row`: global index on the 128-row side; `col0`: global index of v[0] on the other side.
@@ -331,13 +346,15 @@ __device__ __forceinline__ void finish_chunk(const GemmParams& p, const float* v
       const int f0 = col0 >> 1;
       __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + static_cast<size_t>(t) * inter + f0;
       float* dst32 = static_cast<float*>(p.out) + static_cast<size_t>(t) * inter + f0;
+      float limit = 0.0f;
+      if constexpr (EXT) limit = unit_limit_of(p, t / kTileX);
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         if (col0 + 16 + i >= N) break;
         float value;
         if constexpr (EXT)
           value = glu_mul(v[i] + (p.bias ? p.bias[col0 + i] : 0.0f), v[16 + i] + (p.bias ? p.bias[col0 + 16 + i] : 0.0f),
-                          p.activation);
+                          p.activation, limit, p.unit_slope);
         else
           value = silu_mul(v[i], v[16 + i]);
         if (p.out_dtype == VIPERA_BF16) dst[i] = __float2bfloat16_rn(value); else dst32[i] = value;
@@ -828,6 +845,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           int use = 0;
           const int row0 = tx * kTileX + warp * 32;
           if (p.epilogue == EPI_SWIGLU) {
+            float limit = 0.0f;
+            if constexpr (EXT) limit = unit_limit_of(p, tx);
             // 128 accumulator columns make 64 outputs = one 128-byte row of bfloat16
 #pragma unroll 1
             for (int c = 0; c < BN; c += 128) {
@@ -852,8 +871,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                   }
 #pragma unroll
                   for (int i = 0; i < 8; ++i)
-                    packed[i] = pack_bf16x2(glu_mul(v[2 * i], v[16 + 2 * i], p.activation),
-                                            glu_mul(v[2 * i + 1], v[16 + 2 * i + 1], p.activation));
+                    packed[i] = pack_bf16x2(glu_mul(v[2 * i], v[16 + 2 * i], p.activation, limit, p.unit_slope),
+                                            glu_mul(v[2 * i + 1], v[16 + 2 * i + 1], p.activation, limit, p.unit_slope));
                 } else {
 #pragma unroll
                   for (int i = 0; i < 8; ++i)
@@ -1634,7 +1653,8 @@ static int launch_pairs(const CUtensorMap& map_x, const CUtensorMap& map_y, cons
 // `rope`: for EPI_ROPE_CACHE, the fields of that ending (the others are filled in here).
 static int run_gemm(const void* A, const void* W, int T, int N, int K, int epilogue, const float* bias, void* out,
                     int out_dtype, float* resid, float* scratch, size_t scratch_bytes, int* status, void* stream,
-                    const GemmParams* rope, int activation = ACT_SILU, const int* tile_group = nullptr, int groups = 1) {
+                    const GemmParams* rope, int activation = ACT_SILU, const int* tile_group = nullptr, int groups = 1,
+                    const float* unit_limit = nullptr, float unit_slope = 0.0f) {
   if (T <= 0) return VIPERA_OK;
   const bool grouped = tile_group != nullptr;
   if (grouped && (groups <= 0 || T % kTileX != 0 || rope != nullptr || epilogue == EPI_RESIDUAL)) return VIPERA_BAD_ARGUMENT;
@@ -1673,6 +1693,8 @@ static int run_gemm(const void* A, const void* W, int T, int N, int K, int epilo
   if (rope) p = *rope;
   p.tile_group = tile_group;
   p.group_stride = N;
+  p.unit_limit = unit_limit;
+  p.unit_slope = unit_slope;
   p.tokens = T;
   p.features = N;
   p.num_k_blocks = plan.num_k_blocks;
@@ -1786,18 +1808,22 @@ VIPERA_API int vipera_gemm_tc_act(const void* A, const void* W, int T, int N, in
 // Grouped: W is [groups, N, K]; A is [T, K] with T a multiple of 128, and rows 128 * i .. 128 * i + 127
 // are multiplied by matrix tile_group[i] (a device table that a kernel ahead in the stream writes).
 // Endings STORE and the gated unit; STORE into bfloat16 with activation ACT_RELU2 applies the square of
-// relu on the way out (a unit without a gate).
+// relu on the way out (a unit without a gate).  ACT_CLAMPED: the gated unit with the bound
+// unit_limit[tile_group[i]] (a device table) and `unit_slope`.
 VIPERA_API int vipera_gemm_tc_grouped(const void* A, const void* W, int T, int N, int K, int groups, const int* tile_group,
-                                      int epilogue, void* out, int out_dtype, int activation, int* status, void* stream) {
+                                      int epilogue, void* out, int out_dtype, int activation, const float* unit_limit,
+                                      float unit_slope, int* status, void* stream) {
   if (epilogue != EPI_STORE && epilogue != EPI_SWIGLU) return VIPERA_BAD_ARGUMENT;
   if (activation == ACT_RELU2) {
     if (epilogue != EPI_STORE || out_dtype != VIPERA_BF16) return VIPERA_BAD_ARGUMENT;
+  } else if (activation == ACT_CLAMPED) {
+    if (epilogue != EPI_SWIGLU || !unit_limit) return VIPERA_BAD_ARGUMENT;
   } else if (activation != ACT_SILU && activation != ACT_GELU_TANH) {
     return VIPERA_BAD_ARGUMENT;
   }
   if (!tile_group) return VIPERA_BAD_ARGUMENT;
   return run_gemm(A, W, T, N, K, epilogue, nullptr, out, out_dtype, nullptr, nullptr, 0, status, stream, nullptr, activation,
-                  tile_group, groups);
+                  tile_group, groups, unit_limit, unit_slope);
 }
 
 // What the q/k/v ending needs beside the product itself (mirrored by the caller).

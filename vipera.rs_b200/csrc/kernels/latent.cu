@@ -7,14 +7,16 @@
 //
 //   qa_h = [U_h^T q_h | rotated q_h] * scale        (latent_absorb_kernel)
 //   s_j  = qa_h . [c_j | kr_j],  p = softmax over the visible j,  l_h = sum_j p_j c_j
-//                                                    (latent_attention_kernel)
+//                                                    (latent_attention_kernel, latent_fold_kernel)
 //   out_h = (V_h l_h) * sigmoid(gate_h)              (latent_expand_kernel)
 //
 // so the keys and values of earlier tokens are never expanded.  Scores, softmax, the sums over
 // keys, the latent's norm and the rotation are 32-bit.  Rotation: values (2i, 2i + 1) of the
 // rotated part (`pairing` 0) or values (i, i + rot/2) (`pairing` 1) turn by the angle whose cosine
 // and sine the tables hold at [position, i].  With a window w > 0 the query at position p sees keys
-// p - w + 1 .. p only; earlier keys' pages may have been given back and are never read.
+// p - w + 1 .. p only; earlier keys' pages may have been given back and are never read.  With a
+// sink per head the softmax's denominator also holds exp(sink_h): a term without a key or a value,
+// which the scale does not touch.
 #include "attention_mma.cuh"
 
 constexpr int kMaxRank = 512;   // latent size
@@ -29,7 +31,10 @@ __device__ __forceinline__ void rot_pair(int pairing, int rot, int i, int& a, in
 // ---------------------------------------------------------------------------------------
 // The step's latents and rotated key parts into their pages.  `proj` [tokens, proj_width] holds
 // the down projection at column kv_off: rank latent values, then rot key values.  One block per
-// token.  k_pool rows are latents [rank], v_pool rows the rotated key parts [rot].
+// token.  k_pool rows are latents [rank], v_pool rows the rotated key parts [rot].  Where the queries
+// come through a latent of their own (q_rank > 0), its pre-norm values are at column cq_off and the
+// block leaves them normed in `cq` [tokens, q_rank], the operand of the product that makes the
+// queries.  kv_off < 0: the layer keeps nothing of its own, only the query latent is normed.
 // ---------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -37,11 +42,21 @@ latent_store_kernel(const float* __restrict__ proj, long long proj_width, int kv
                     float eps, const int* __restrict__ positions, const float* __restrict__ cos_table,
                     const float* __restrict__ sin_table, T* __restrict__ k_pool, T* __restrict__ v_pool,
                     const int* __restrict__ token_entry, const int* __restrict__ block_table, int table_width,
-                    int page_size, int rank, int rot, int pairing) {
+                    int page_size, int rank, int rot, int pairing, int cq_off, int q_rank,
+                    const float* __restrict__ cq_norm_weight, T* __restrict__ cq) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
+  if (q_rank > 0) {
+    const float* q_row = proj + static_cast<size_t>(t) * proj_width + cq_off;
+    float squares = 0.0f;
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) squares += q_row[i] * q_row[i];
+    const float inverse = 1.0f / sqrtf(block_sum(squares, scratch) / static_cast<float>(q_rank) + eps);
+    T* dst = cq + static_cast<size_t>(t) * q_rank;
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) dst[i] = from_float<T>(q_row[i] * inverse * cq_norm_weight[i]);
+  }
+  if (kv_off < 0) return;
   const float* row = proj + static_cast<size_t>(t) * proj_width + kv_off;
   const int position = positions[t];
   const int page = block_table[static_cast<size_t>(token_entry[t]) * table_width + position / page_size];
@@ -174,7 +189,7 @@ __global__ void __launch_bounds__(kWarps * 32)
 latent_attention_kernel(const float* __restrict__ qa, float* __restrict__ mixed, const T* __restrict__ k_pool,
                         const T* __restrict__ v_pool, const int* __restrict__ token_entry,
                         const int* __restrict__ positions, const int* __restrict__ block_table, int table_width,
-                        int page_size, int heads, int rank, int rot, int window) {
+                        int page_size, int heads, int rank, int rot, int window, const float* __restrict__ sink) {
   extern __shared__ float q_shared[];   // [kWarps][rank + rot]
   pdl_launch_dependents();
   pdl_wait();
@@ -221,6 +236,10 @@ latent_attention_kernel(const float* __restrict__ qa, float* __restrict__ mixed,
       }
     }
   }
+  if (sink) {
+    // where the sink is far above every score the quotient is 0, as it should be
+    running_sum += expf(sink[h] - running_max);
+  }
   const float inverse = 1.0f / running_sum;
   float* out_row = mixed + (static_cast<size_t>(t) * heads + h) * rank;
 #pragma unroll
@@ -239,8 +258,10 @@ latent_attention_kernel(const float* __restrict__ qa, float* __restrict__ mixed,
 //   1. each score 8 keys against all 16 rows: S = Q K^T over rank + rot values;
 //   2. each take two rows: running maximum, weights p = exp(s - m) rounded to bfloat16, their sum;
 //   3. each add P C into their 1/8 of the latent's columns.
-// With `num_splits` > 1 a block folds keys [split * split_keys, ...) only and leaves (m, sum,
-// unnormalised columns); latent_combine_kernel joins the splits.  NR: the columns the block's
+// With `num_splits` > 1 a block folds `split_keys` keys only and leaves (m, sum, unnormalised
+// columns); latent_combine_kernel joins the splits.  The splits are counted from key 0 or, with a
+// window, from the tile of 64 keys that holds the first key the pass's rows see (so a long history
+// costs a windowed step no more than the window).  NR: the columns the block's
 // accumulators cover (128, 256 or 512, at least the rank rounded up to 16).
 // ---------------------------------------------------------------------------------------
 constexpr int kFoldRows = 16;
@@ -261,6 +282,7 @@ struct LatentFoldParams {
   int num_tokens, heads, rank, rot, table_width, page_size;
   int head_group, tokens_per_tile, split_keys, num_splits;
   int window;                      // > 0: a row at position p sees keys p - window + 1 .. p
+  const float* sink;               // [heads] or null: exp(sink_h) joins the softmax's denominator
   // Head-major form (the products on both sides of the fold run as grouped tensor-core products, a
   // head a group): the unrotated part of qa comes unscaled from qa_heads [heads, padded_tokens, rank]
   // and the rotated, scaled part from q_rot [tokens, heads, rot]; the folded latents leave as
@@ -349,11 +371,9 @@ latent_fold_kernel(LatentFoldParams p) {
       }
       q_s[r * stride + (c < p.rank ? c : rank_pad + c - p.rank)] = __float2bfloat16(v);
     }
-    // tiles are counted from the split's first key, whatever the window: the first tile that holds a
-    // visible key is the first one folded
-    const int split_begin = split * p.split_keys;
-    const int begin = split_begin + max(0, first_key - split_begin) / kFoldKeys * kFoldKeys;
-    const int end = min(last_key + 1, split_begin + p.split_keys);
+    // first_key is 0 without a window; tiles start at multiples of kFoldKeys either way
+    const int begin = first_key / kFoldKeys * kFoldKeys + split * p.split_keys;
+    const int end = p.num_splits > 1 ? min(last_key + 1, begin + p.split_keys) : last_key + 1;
     const int num_tiles = end > begin ? (end - begin + kFoldKeys - 1) / kFoldKeys : 0;
     const int* table = p.block_table + static_cast<size_t>(entry) * p.table_width;
 
@@ -493,7 +513,8 @@ latent_fold_kernel(LatentFoldParams p) {
       const int row = mt * kFoldRows + g + half * 8;
       const int out_row = row_s[row];
       if (out_row < 0) continue;
-      const float total = l_s[row];
+      float total = l_s[row];
+      if (p.sink && p.num_splits == 1) total += expf(p.sink[out_row % p.heads] - m_s[row]);
       if (p.num_splits == 1 && p.l_heads != nullptr) {
         const float inverse = 1.0f / total;
         __nv_bfloat16* l_row = p.l_heads + (static_cast<size_t>(out_row % p.heads) * p.padded_tokens + out_row / p.heads) * p.rank;
@@ -555,6 +576,7 @@ latent_combine_kernel(LatentFoldParams p) {
       weight_s[s] = sum_s[s] > 0.0f ? expf(top_s[s] - top) : 0.0f;
       total += sum_s[s] * weight_s[s];
     }
+    if (p.sink) total += expf(p.sink[row % p.heads] - top);
     const float inverse = 1.0f / total;
     for (int s = 0; s < p.num_splits; ++s) weight_s[s] *= inverse;
   }
@@ -718,6 +740,15 @@ struct LatentParams {
   int* tile_group;         // [heads * padded_tokens / 128]
   int window;              // > 0: a query at position p sees keys p - window + 1 .. p
   int pairing;             // of the rotated part: 0 values (2i, 2i + 1), 1 values (i, i + rot/2)
+  const float* sink;       // [heads] or null
+  // Queries that are no columns of `proj`: [tokens, q_width], at column q_off (null: in `proj`).
+  const float* q;
+  long long q_width;
+  // stage 4 (ahead of the product that makes such queries): the cache write as above and, with
+  // q_rank > 0, the normed query latent.
+  int cq_off, q_rank;
+  const float* cq_norm_weight;   // [q_rank]
+  void* cq;                      // [tokens, q_rank], the run's type
 };
 
 // How the tensor-core fold cuts a step: {tokens per tile, heads per tile, keys per split, splits}.
@@ -731,10 +762,13 @@ static int fold_groups(int tokens, int heads, int sms) {
   return base >= 2L * sms && heads <= kFoldRows ? 2 : 1;
 }
 
-static void latent_plan(int tokens, int heads, int max_keys, int sms, int* plan) {
+static void latent_plan(int tokens, int heads, int max_keys, int window, int sms, int* plan) {
   const int head_group = heads < kFoldRows ? heads : kFoldRows;
   const int per_tile = kFoldRows * fold_groups(tokens, heads, sms) / head_group;
   const long base = static_cast<long>((tokens + per_tile - 1) / per_tile) * ((heads + head_group - 1) / head_group);
+  // with a window a tile's rows together see window + per_tile - 1 keys at most, counted from the
+  // start of a tile of keys
+  if (window > 0 && max_keys > window + per_tile + kFoldKeys) max_keys = window + per_tile + kFoldKeys;
   int bound = kFoldKeys;
   while (bound < max_keys) bound *= 2;
   long want = (4L * sms) / base;
@@ -749,9 +783,9 @@ static void latent_plan(int tokens, int heads, int max_keys, int sms, int* plan)
   plan[3] = (bound + chunk - 1) / chunk;
 }
 
-VIPERA_API int vipera_latent_plan(int tokens, int heads, int max_keys, int sms, int* plan) {
-  if (tokens <= 0 || heads <= 0 || sms <= 0) return VIPERA_BAD_ARGUMENT;
-  latent_plan(tokens, heads, max_keys < 1 ? 1 : max_keys, sms, plan);
+VIPERA_API int vipera_latent_plan(int tokens, int heads, int max_keys, int window, int sms, int* plan) {
+  if (tokens <= 0 || heads <= 0 || sms <= 0 || window < 0) return VIPERA_BAD_ARGUMENT;
+  latent_plan(tokens, heads, max_keys < 1 ? 1 : max_keys, window, sms, plan);
   return VIPERA_OK;
 }
 
@@ -779,6 +813,7 @@ static int launch_fold_any(const LatentParams& p, cudaStream_t s) {
   f.num_tokens = p.num_tokens, f.heads = p.heads, f.rank = p.rank, f.rot = p.rot;
   f.table_width = p.table_width, f.page_size = p.page_size;
   f.window = p.window;
+  f.sink = p.sink;
   if (p.stage == 2) {
     f.qa_heads = p.qa_heads, f.q_rot = p.q_rot, f.l_heads = static_cast<__nv_bfloat16*>(p.l_heads);
     f.padded_tokens = p.padded_tokens, f.scale = p.scale;
@@ -819,20 +854,22 @@ static int launch_latent(const LatentParams& p, cudaStream_t s) {
     return vipera_launch(latent_gate_kernel<T>, static_cast<unsigned>((values + 255) / 256), 256, 0, s, p.o_heads, p.proj,
                          p.proj_width, p.g_off, static_cast<T*>(p.out), p.num_tokens, p.heads, p.dv, p.padded_tokens);
   }
-  if (p.kv_off >= 0) {
+  if (p.kv_off >= 0 || p.stage == 4) {
     status = vipera_launch(latent_store_kernel<T>, p.num_tokens, 128, 0, s, p.proj, p.proj_width, p.kv_off, p.norm_weight,
                            p.eps, p.positions, p.cos_table, p.sin_table, static_cast<T*>(p.k_pool),
                            static_cast<T*>(p.v_pool), p.token_entry, p.block_table, p.table_width, p.page_size, p.rank,
-                           p.rot, p.pairing);
-    if (status) return status;
+                           p.rot, p.pairing, p.cq_off, p.stage == 4 ? p.q_rank : 0, p.cq_norm_weight, static_cast<T*>(p.cq));
+    if (status || p.stage == 4) return status;
   }
+  const float* q = p.q ? p.q : p.proj;
+  const long long q_width = p.q ? p.q_width : p.proj_width;
   if (p.stage == 1)
-    return vipera_launch(latent_prep_kernel, p.num_tokens, 128, 0, s, p.proj, p.proj_width, p.q_off, p.positions, p.cos_table,
+    return vipera_launch(latent_prep_kernel, p.num_tokens, 128, 0, s, q, q_width, p.q_off, p.positions, p.cos_table,
                          p.sin_table, static_cast<__nv_bfloat16*>(p.a_heads), p.q_rot, p.tile_group, p.heads, p.d, p.rot,
                          p.padded_tokens, p.scale, p.pairing);
   const dim3 tiles((p.num_tokens + kTile - 1) / kTile, p.heads);
   const dim3 absorb_grid(tiles.x, tiles.y, (p.rank + 127) / 128);
-  status = vipera_launch(latent_absorb_kernel<T>, absorb_grid, 128, kTile * p.d * sizeof(float), s, p.proj, p.proj_width, p.q_off,
+  status = vipera_launch(latent_absorb_kernel<T>, absorb_grid, 128, kTile * p.d * sizeof(float), s, q, q_width, p.q_off,
                          static_cast<const T*>(p.up_k), p.positions, p.cos_table, p.sin_table, p.qa, p.num_tokens,
                          p.heads, p.d, p.rank, p.rot, p.scale, p.pairing);
   if (status) return status;
@@ -844,7 +881,7 @@ static int launch_latent(const LatentParams& p, cudaStream_t s) {
     status = vipera_launch(latent_attention_kernel<T>, dim3(p.num_tokens, (p.heads + kWarps - 1) / kWarps), kWarps * 32,
                            kWarps * (p.rank + p.rot) * sizeof(float), s, p.qa, p.latent_out,
                            static_cast<const T*>(p.k_pool), static_cast<const T*>(p.v_pool), p.token_entry, p.positions,
-                           p.block_table, p.table_width, p.page_size, p.heads, p.rank, p.rot, p.window);
+                           p.block_table, p.table_width, p.page_size, p.heads, p.rank, p.rot, p.window, p.sink);
   if (status) return status;
   const dim3 expand_grid(tiles.x, tiles.y, (p.dv + 31) / 32);
   return vipera_launch(latent_expand_kernel<T, T>, expand_grid, 128, (kTile * p.rank + 4 * kTile * 32) * sizeof(float), s, p.latent_out,
@@ -859,8 +896,12 @@ VIPERA_API int vipera_latent_attention(const LatentParams* params, int dtype, vo
   if (p.rank <= 0 || p.rank > kMaxRank || p.rot <= 0 || p.rot > kMaxRot || (p.rot & 1)) return VIPERA_BAD_SHAPE;
   if (p.heads <= 0 || p.d <= 0 || p.d > 1024 || p.dv <= 0 || p.page_size <= 0 || p.table_width <= 0) return VIPERA_BAD_SHAPE;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (p.stage < 0 || p.stage > 3 || p.window < 0 || p.pairing < 0 || p.pairing > 1) return VIPERA_BAD_ARGUMENT;
-  if (p.stage != 0) {
+  if (p.stage < 0 || p.stage > 4 || p.window < 0 || p.pairing < 0 || p.pairing > 1) return VIPERA_BAD_ARGUMENT;
+  if (p.q && p.q_width < static_cast<long long>(p.q_off) + static_cast<long long>(p.heads) * (p.d + p.rot)) return VIPERA_BAD_SHAPE;
+  if (p.stage == 4) {
+    if (p.q_rank < 0 || (p.q_rank > 0 && (!p.cq || !p.cq_norm_weight || p.cq_off < 0 || p.cq_off + p.q_rank > p.proj_width)))
+      return VIPERA_BAD_ARGUMENT;
+  } else if (p.stage != 0) {
     if (dtype != VIPERA_BF16 || p.rank % 8 || p.rot % 8 || p.d % 8 || p.padded_tokens < p.num_tokens || p.padded_tokens % 128 ||
         !p.a_heads || !p.qa_heads || !p.q_rot || !p.l_heads || !p.o_heads || !p.tile_group ||
         p.num_tokens >= (1 << 24) / p.heads || (p.num_splits > 1 && p.split_keys % kFoldKeys))

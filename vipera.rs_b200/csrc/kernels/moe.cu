@@ -1,7 +1,7 @@
 // A mixture of gated feed-forward units: router, grouping of the step's (token, expert)
 // assignments by expert, and the experts' products over tiles of assignments.
 //
-//   z = R h (32-bit), s = sigmoid(z) or softmax(z)
+//   z = R h (32-bit), s = sigmoid(z), softmax(z) or z itself
 //   experts in `groups` equal groups of neighbours; a group's score is the sum of its `group_top`
 //   largest scores; only experts of the `keep` best groups may be chosen; the `top` largest
 //   scores among those are the token's experts, with weights s (divided by their sum if asked).
@@ -32,7 +32,11 @@
 // row).  `always`: that many units beyond the router's own which every token uses with weight 1 (a
 // shared unit, cut into pieces of the experts' inner size); their matrices follow the chosen experts'
 // in the same tensors, and a token has `slots` = top + always assignments.  With `renormalize` the
-// weights are divided by their sum + `renorm_eps`; `route_scale` multiplies them.
+// weights are divided by their sum + `renorm_eps`; `route_scale` multiplies them.  Scores that are the
+// logits themselves (`scores` 2): the weights are the softmax over the chosen logits only.
+// `always_gate`: the router's matrix has one row more, and the always-used units' weight is the
+// sigmoid of that row's product with h.  ACT_CLAMPED: a gated unit with bounds (`unit_limit`, one per
+// unit with matrices) and the slope `unit_slope` inside its sigmoid.
 #include "common.cuh"
 
 constexpr int kTileRows = 32;
@@ -44,7 +48,7 @@ constexpr int kRouteThreads = 256;
 
 struct MoeParams {
   const void* h;            // [tokens, hidden], the run's type
-  const float* router;      // [experts, hidden]
+  const float* router;      // [experts (+ 1 with always_gate), hidden]
   const void* gate_up;      // [experts, 2 ff, hidden]
   const void* down;         // [experts, hidden, ff]
   int* chosen;              // [tokens * top]
@@ -58,7 +62,8 @@ struct MoeParams {
   void* xs;                 // padded form: [capacity, hidden] the tokens' rows in sorted order
   float* ys;                // padded form: [capacity, hidden] the down products in sorted order
   int num_tokens, hidden, ff, experts, top, groups, keep, group_top, max_tiles;
-  int softmax_scores, renormalize, activation;
+  int scores;               // 0: sigmoid(z), 1: softmax(z), 2: z, weighted by the softmax over the chosen
+  int renormalize, activation;
   int gate_group;           // gate rows and up rows alternate in groups of this many
   int tile_rows;            // 8, 32 or (padded) 128
   int padded;               // 1: every expert's run starts at a multiple of tile_rows; capacity = max_tiles * tile_rows
@@ -68,7 +73,16 @@ struct MoeParams {
   int slots;                // top + always: a token's assignments
   int gated;                // 1: gated units; 0: act(U h)
   float route_scale, renorm_eps;
+  int always_gate;          // 1: the always-used units' weight is sigmoid(the router's last row . h)
+  const float* unit_limit;  // ACT_CLAMPED: [matrices]
+  float unit_slope;
 };
+
+// The gated unit of matrix `unit`.
+__device__ __forceinline__ float moe_gated(const MoeParams& p, float gate, float up, int unit) {
+  if (p.activation == ACT_CLAMPED) return clamped_unit(gate, up, p.unit_limit[unit], p.unit_slope);
+  return gate_activation(gate, p.activation) * up;
+}
 
 // The units that have matrices: the router's outputs without the identity ones, then the ones every token uses.
 __device__ __forceinline__ int moe_matrices(const MoeParams& p) { return p.experts - p.identity + p.always; }
@@ -101,8 +115,9 @@ moe_route_kernel(MoeParams p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
   float* h_s = route_shared;                // [hidden] (first: read as vectors)
+  const int rows_total = p.experts + p.always_gate;
   float* score = h_s + p.hidden;
-  float* open = score + p.experts;          // the score while the expert may still be chosen, else -inf
+  float* open = score + rows_total;         // the score while the expert may still be chosen, else -inf
   float* group_score = open + p.experts;
   const T* h = static_cast<const T*>(p.h) + static_cast<size_t>(t) * p.hidden;
   for (int i = threadIdx.x; i < p.hidden; i += kRouteThreads) h_s[i] = to_float<T>(h[i]);
@@ -113,12 +128,12 @@ moe_route_kernel(MoeParams p) {
     // walks four of its rows side by side, so that their loads are in flight together (a step of one token is
     // one block, which waits for every row it asks for).
     const float4* h4 = reinterpret_cast<const float4*>(h_s);
-    for (int e0 = warp; e0 < p.experts; e0 += 4 * kWarpsHere) {
+    for (int e0 = warp; e0 < rows_total; e0 += 4 * kWarpsHere) {
       const float4* rows[4];
       float sums[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
       for (int j = 0; j < 4; ++j)
-        rows[j] = reinterpret_cast<const float4*>(p.router + static_cast<size_t>(min(e0 + j * kWarpsHere, p.experts - 1)) * p.hidden);
+        rows[j] = reinterpret_cast<const float4*>(p.router + static_cast<size_t>(min(e0 + j * kWarpsHere, rows_total - 1)) * p.hidden);
 #pragma unroll 4
       for (int i = lane; i < p.hidden / 4; i += 32) {
         const float4 a = h4[i];
@@ -136,11 +151,11 @@ moe_route_kernel(MoeParams p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const float sum = warp_sum(sums[j]);
-        if (lane == 0 && e0 + j * kWarpsHere < p.experts) score[e0 + j * kWarpsHere] = sum;
+        if (lane == 0 && e0 + j * kWarpsHere < rows_total) score[e0 + j * kWarpsHere] = sum;
       }
     }
   } else {
-    for (int e = warp; e < p.experts; e += kWarpsHere) {
+    for (int e = warp; e < rows_total; e += kWarpsHere) {
       const float* r = p.router + static_cast<size_t>(e) * p.hidden;
       float sum = 0.0f;
 #pragma unroll 4
@@ -151,7 +166,7 @@ moe_route_kernel(MoeParams p) {
   }
   __syncthreads();
   if (warp == 0) {
-  if (p.softmax_scores) {
+  if (p.scores == 1) {
     float top_z = -INFINITY;
     for (int e = lane; e < p.experts; e += 32) top_z = fmaxf(top_z, score[e]);
     top_z = warp_max(top_z);
@@ -159,7 +174,7 @@ moe_route_kernel(MoeParams p) {
     for (int e = lane; e < p.experts; e += 32) total += expf(score[e] - top_z);
     total = warp_sum(total);
     for (int e = lane; e < p.experts; e += 32) score[e] = expf(score[e] - top_z) / total;
-  } else {
+  } else if (p.scores == 0) {
     for (int e = lane; e < p.experts; e += 32) score[e] = 1.0f / (1.0f + expf(-score[e]));
   }
   __syncwarp();
@@ -205,7 +220,7 @@ moe_route_kernel(MoeParams p) {
       if (group_score[e / per_group] != INFINITY) open[e] = -INFINITY;
     __syncwarp();
   }
-  float total = 0.0f;
+  float total = 0.0f, first_z = 0.0f;
   for (int place = 0; place < p.top; ++place) {
     float best = -INFINITY;
     int at = 0x7fffffff;
@@ -215,7 +230,11 @@ moe_route_kernel(MoeParams p) {
     }
     warp_argmax(best, at);
     if (at == 0x7fffffff) at = 0;   // cannot happen with top <= keep * per_group; keeps the index in range
-    const float w = score[at];
+    float w = score[at];
+    if (p.scores == 2) {   // (the first chosen logit is the largest unless a correction chose otherwise)
+      if (place == 0) first_z = w;
+      w = expf(w - first_z);
+    }
     total += w;
     if (lane == 0) {
       // an output without matrices is marked -1 - (its index among those)
@@ -226,14 +245,15 @@ moe_route_kernel(MoeParams p) {
     __syncwarp();
   }
   if (lane == 0) {
-    const float divisor = p.renormalize ? total + p.renorm_eps : 1.0f;
+    const float divisor = p.scores == 2 ? total : p.renormalize ? total + p.renorm_eps : 1.0f;
+    const float always_weight = p.always_gate ? 1.0f / (1.0f + expf(-score[p.experts])) : 1.0f;
     for (int place = 0; place < p.top; ++place) {
       const size_t a = static_cast<size_t>(t) * p.slots + place;
       p.weight[a] = p.weight[a] / divisor * p.route_scale;
     }
     for (int extra = 0; extra < p.always; ++extra) {
       p.chosen[static_cast<size_t>(t) * p.slots + p.top + extra] = p.experts - p.identity + extra;
-      p.weight[static_cast<size_t>(t) * p.slots + p.top + extra] = 1.0f;
+      p.weight[static_cast<size_t>(t) * p.slots + p.top + extra] = always_weight;
     }
   }
   }
@@ -425,7 +445,7 @@ moe_skinny_kernel(MoeParams p) {
       for (int f = 0; f < 2; ++f)
         if (col0 + f < outer)
           static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + col0 + f] =
-              from_float<T>(gate_activation(acc[2 * f][r], p.activation) * acc[2 * f + 1][r]);
+              from_float<T>(moe_gated(p, acc[2 * f][r], acc[2 * f + 1][r], expert));
     } else if (FIRST) {
 #pragma unroll
       for (int j = 0; j < 4; ++j)
@@ -520,7 +540,7 @@ moe_product_kernel(MoeParams p) {
       if (c >= outer) continue;
       if (GATED) {
         static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + c] =
-            from_float<T>(gate_activation(acc0[i][j], p.activation) * acc1[i][j]);
+            from_float<T>(moe_gated(p, acc0[i][j], acc1[i][j], expert));
       } else if (FIRST) {
         static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + c] = from_float<T>(gate_activation(acc0[i][j], p.activation));
       } else {
@@ -563,7 +583,7 @@ static int launch_skinny(const MoeParams& p, cudaStream_t s) {
 // The router, the grouping and (padded form) the gathered rows.
 template <typename T>
 static int launch_route(const MoeParams& p, cudaStream_t s) {
-  const size_t route_shared = static_cast<size_t>(2 * p.experts + p.groups + p.hidden) * sizeof(float);
+  const size_t route_shared = static_cast<size_t>(2 * p.experts + p.always_gate + p.groups + p.hidden) * sizeof(float);
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(moe_route_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
@@ -602,7 +622,9 @@ static int check_moe(const MoeParams& p) {
   if (p.max_tiles < p.num_tokens * p.slots / p.tile_rows + min(p.experts - p.identity + p.always, p.num_tokens * p.slots) ||
       p.max_tiles > 65535)
     return VIPERA_BAD_ARGUMENT;
-  if (static_cast<size_t>(2 * p.experts + p.groups + p.hidden) * sizeof(float) > 200 * 1024) return VIPERA_BAD_SHAPE;
+  if (p.scores < 0 || p.scores > 2 || p.always_gate < 0 || p.always_gate > 1) return VIPERA_BAD_ARGUMENT;
+  if (p.activation == ACT_CLAMPED && (!p.gated || !p.unit_limit)) return VIPERA_BAD_ARGUMENT;
+  if (static_cast<size_t>(2 * p.experts + p.always_gate + p.groups + p.hidden) * sizeof(float) > 200 * 1024) return VIPERA_BAD_SHAPE;
   if (p.tile_rows == kSkinnyRows && static_cast<size_t>(kSkinnyRows) * max(p.hidden, p.ff) * 4 > 200 * 1024) return VIPERA_BAD_SHAPE;
   if (p.padded && (!p.xs || !p.ys || (p.hidden * 2) % 16 || (reinterpret_cast<uintptr_t>(p.xs) & 15) ||
                    (reinterpret_cast<uintptr_t>(p.h) & 15) || (reinterpret_cast<uintptr_t>(p.ys) & 15) ||

@@ -277,3 +277,166 @@ VIPERA_API int vipera_layernorm(const float* x, const float* weight, const float
 }
 
 VIPERA_API const char* vipera_rowwise_status_text(int status) { return vipera_status_text(status); }
+
+// ---------------------------------------------------------------------------------------
+// Branches computed from one and the same stream join it, and the norms that read the result next
+// follow in the same pass over the row:
+//   x += scale_a * (sum of a's parts) + scale_b * (sum of b's parts)
+//   out1 = norm1(x), out2 = norm2(x)                      (RMS norms, 32-bit statistics)
+// A branch is [rows, parts, hidden] (its parts added in their order), its scale one number per
+// channel or null; either branch and either norm may be missing.  With `rows` the kernel computes
+// norms of the rows named there and leaves x as it is.  A block per row; VEC values to an access; the
+// row stays in registers between its passes where it is short enough.
+// ---------------------------------------------------------------------------------------
+struct JoinBranch {
+  const float* values;   // null: no such branch
+  const float* scale;    // [hidden] or null: 1
+  int parts;
+};
+struct JoinNorm {
+  const float* gain;     // null: no such norm
+  void* out;             // [rows, hidden]
+  float eps;
+};
+struct JoinParams {
+  float* x;
+  const int* rows;
+  JoinBranch branch[2];
+  JoinNorm norm[2];
+  int num_rows, hidden, out_dtype;
+};
+
+template <int VEC>
+struct JoinVector { float v[VEC]; };
+
+template <int VEC>
+__device__ __forceinline__ JoinVector<VEC> join_load(const float* src) {
+  JoinVector<VEC> r;
+  if constexpr (VEC == 4) {
+    const float4 q = *reinterpret_cast<const float4*>(src);
+    r.v[0] = q.x, r.v[1] = q.y, r.v[2] = q.z, r.v[3] = q.w;
+  } else {
+    r.v[0] = *src;
+  }
+  return r;
+}
+
+template <typename TO, int VEC>
+__device__ __forceinline__ void join_store(TO* dst, const JoinVector<VEC>& a) {
+  if constexpr (VEC == 4) store_four(dst, a.v[0], a.v[1], a.v[2], a.v[3]);
+  else *dst = from_float<TO>(a.v[0]);
+}
+
+// The branch's share of values i .. i + VEC - 1 of a row, added to `to`.
+template <int VEC>
+__device__ __forceinline__ void join_add(JoinVector<VEC>& to, const JoinBranch& b, size_t row, int hidden, int i) {
+  if (!b.values) return;
+  const float* src = b.values + row * b.parts * hidden + i;
+  JoinVector<VEC> sum = join_load<VEC>(src);
+#pragma unroll 4
+  for (int p = 1; p < b.parts; ++p) {
+    const JoinVector<VEC> more = join_load<VEC>(src + static_cast<size_t>(p) * hidden);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) sum.v[e] += more.v[e];
+  }
+  if (b.scale) {
+    const JoinVector<VEC> s = join_load<VEC>(b.scale + i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) to.v[e] = fmaf(s.v[e], sum.v[e], to.v[e]);
+  } else {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) to.v[e] += sum.v[e];
+  }
+}
+
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(kNormThreads)
+join_norms_kernel(const JoinParams p) {
+  __shared__ float scratch[32];
+  constexpr int kKept = VEC == 4 ? 4 : 8;   // vectors a thread keeps: rows up to 4096 (2048) wide
+  pdl_launch_dependents();
+  const int r = blockIdx.x;
+  const int first = threadIdx.x * VEC, step = kNormThreads * VEC;
+  const bool fits = p.hidden <= kKept * step;
+  pdl_wait();
+  const size_t row = p.rows ? p.rows[r] : r;
+  float* x = p.x + row * p.hidden;
+  JoinVector<VEC> kept[kKept];
+  float squares = 0.0f;
+  auto joined = [&](int i) {
+    JoinVector<VEC> v = join_load<VEC>(x + i);
+    join_add<VEC>(v, p.branch[0], row, p.hidden, i);
+    join_add<VEC>(v, p.branch[1], row, p.hidden, i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) squares = fmaf(v.v[e], v.v[e], squares);
+    return v;
+  };
+  const bool writes = p.rows == nullptr && (p.branch[0].values || p.branch[1].values);
+  if (fits) {
+#pragma unroll
+    for (int j = 0; j < kKept; ++j) {
+      const int i = first + j * step;
+      if (i < p.hidden) {
+        kept[j] = joined(i);
+        if (writes) join_store<float, VEC>(x + i, kept[j]);
+      }
+    }
+  } else {
+    for (int i = first; i < p.hidden; i += step) {
+      const JoinVector<VEC> v = joined(i);
+      if (writes) join_store<float, VEC>(x + i, v);
+    }
+  }
+  if (!p.norm[0].gain && !p.norm[1].gain) return;
+  const float mean = block_sum(squares, scratch) / static_cast<float>(p.hidden);
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    const JoinNorm& norm = p.norm[n];
+    if (!norm.gain) continue;
+    const float inverse = 1.0f / sqrtf(mean + norm.eps);
+    TO* out = static_cast<TO*>(norm.out) + static_cast<size_t>(r) * p.hidden;
+    auto finish = [&](JoinVector<VEC> v, int i) {
+      const JoinVector<VEC> g = join_load<VEC>(norm.gain + i);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v.v[e] = v.v[e] * inverse * g.v[e];
+      join_store<TO, VEC>(out + i, v);
+    };
+    if (fits) {
+#pragma unroll
+      for (int j = 0; j < kKept; ++j) {
+        const int i = first + j * step;
+        if (i < p.hidden) finish(kept[j], i);
+      }
+    } else {
+      // a thread reads back what it wrote itself; with `rows` nothing was written and the sum is formed again
+      for (int i = first; i < p.hidden; i += step) finish(writes || (!p.branch[0].values && !p.branch[1].values) ? join_load<VEC>(x + i) : joined(i), i);
+    }
+  }
+}
+
+template <typename TO>
+static int launch_join(const JoinParams& p, bool vectors, cudaStream_t s) {
+  if (vectors) return vipera_launch(join_norms_kernel<TO, 4>, p.num_rows, kNormThreads, 0, s, p);
+  return vipera_launch(join_norms_kernel<TO, 1>, p.num_rows, kNormThreads, 0, s, p);
+}
+
+// out_dtype: the type of both norms' outputs.
+VIPERA_API int vipera_join_norms(const JoinParams* params, void* stream) {
+  const JoinParams& p = *params;
+  if (p.num_rows <= 0) return VIPERA_OK;
+  if (p.hidden <= 0 || !p.x) return VIPERA_BAD_SHAPE;
+  uintptr_t bases = reinterpret_cast<uintptr_t>(p.x);
+  for (int i = 0; i < 2; ++i) {
+    if (p.branch[i].values && p.branch[i].parts <= 0) return VIPERA_BAD_ARGUMENT;
+    if (p.norm[i].gain && !p.norm[i].out) return VIPERA_BAD_ARGUMENT;
+    bases |= reinterpret_cast<uintptr_t>(p.branch[i].values) | reinterpret_cast<uintptr_t>(p.branch[i].scale) |
+             reinterpret_cast<uintptr_t>(p.norm[i].gain) | reinterpret_cast<uintptr_t>(p.norm[i].out);
+  }
+  const bool vectors = p.hidden % 4 == 0 && (bases & 15) == 0;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (p.out_dtype == VIPERA_F32) return launch_join<float>(p, vectors, s);
+  if (p.out_dtype == VIPERA_BF16) return launch_join<__nv_bfloat16>(p, vectors, s);
+  return VIPERA_BAD_DTYPE;
+}
+
+VIPERA_API int vipera_join_params_size() { return static_cast<int>(sizeof(JoinParams)); }

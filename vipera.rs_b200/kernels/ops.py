@@ -20,8 +20,9 @@ from ..errors import InternalError, InvalidArgumentError, UnsupportedError
 F32, BF16 = 0, 1
 EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU = 0, 1, 2
 EPI_GATED = EPI_SWIGLU   # the gated unit over interleaved gate and up rows; its activation is an argument
-ACT_SILU, ACT_GELU_TANH, ACT_RELU2 = 0, 1, 2
+ACT_SILU, ACT_GELU_TANH, ACT_RELU2, ACT_CLAMPED = 0, 1, 2, 3
 ACTIVATIONS = {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH}   # of a gated unit's gate
+BOUNDED_ACTIVATIONS = {**ACTIVATIONS, "clamped": ACT_CLAMPED}   # of an expert (clamped: both halves of the unit have bounds)
 UNIT_ACTIVATIONS = {**ACTIVATIONS, "relu2": ACT_RELU2}          # of a unit without a gate (relu2: the square of relu)
 ROPE_NONE, ROPE_NEOX, ROPE_INTERLEAVED = 0, 1, 2
 SAMPLE_OK, SAMPLE_NO_FINITE, SAMPLE_NO_MASS, SAMPLE_NEEDS_HOST = 0, 1, 2, 3
@@ -231,6 +232,46 @@ def sm_count(device) -> int:
     if count is None:
         count = _sm_counts[key] = int(torch.cuda.get_device_properties(device).multi_processor_count)
     return count
+
+
+class _JoinBranch(ctypes.Structure):
+    _fields_ = [("values", _c_void), ("scale", _c_void), ("parts", _c_int)]
+
+
+class _JoinNorm(ctypes.Structure):
+    _fields_ = [("gain", _c_void), ("out", _c_void), ("eps", _c_float)]
+
+
+class _JoinParams(ctypes.Structure):
+    _fields_ = [("x", _c_void), ("rows", _c_void), ("branch", _JoinBranch * 2), ("norm", _JoinNorm * 2),
+                ("num_rows", _c_int), ("hidden", _c_int), ("out_dtype", _c_int)]
+
+
+def join_norms(x: torch.Tensor, branches=(), norms=(), rows: Optional[torch.Tensor] = None) -> None:
+    """Up to two branches join the float32 stream ``x`` [rows, hidden] and up to two RMS norms read the
+    result.  A branch is ``(values, parts, scale)``: ``x += scale * sum over the parts`` with values float32
+    [rows, parts * hidden] and scale float32 [hidden] or None.  A norm is ``(gain, eps, out)``.  With
+    ``rows`` (int32) the norms are those of the rows named there, and x stays as it is."""
+    fn = _function("rowwise", "vipera_join_norms", [ctypes.POINTER(_JoinParams), _c_void])
+    _check_struct("rowwise", "vipera_join_params_size", _JoinParams)
+    hidden = x.shape[-1]
+    count = x.numel() // hidden if rows is None else rows.numel()
+    if len(branches) > 2 or len(norms) > 2 or not (branches or norms) or (rows is not None and not norms):
+        raise InvalidArgumentError("join_norms: up to two branches and up to two norms, at least one of them")
+    p = _JoinParams()
+    p.x, p.rows = _gpu(x, "x", torch.float32), _opt(rows, "rows", torch.int32)
+    p.num_rows, p.hidden = count, hidden
+    for slot, (values, parts, scale) in zip(p.branch, branches):
+        if values.numel() != x.numel() * int(parts) or (scale is not None and scale.numel() != hidden):
+            raise InvalidArgumentError("join_norms: a branch holds parts rows of the stream's width per row, its scale one "
+                                       "number per channel")
+        slot.values, slot.scale, slot.parts = _gpu(values, "values", torch.float32), _opt(scale, "scale", torch.float32), int(parts)
+    for slot, (gain, eps, out) in zip(p.norm, norms):
+        if gain.numel() != hidden or out.numel() != count * hidden or out.dtype != norms[0][2].dtype:
+            raise InvalidArgumentError("join_norms: a norm's gain is [hidden] and its output [rows, hidden], all of one type")
+        slot.gain, slot.eps, slot.out = _gpu(gain, "gain", torch.float32), float(eps), _gpu(out, "out")
+    p.out_dtype = dtype_code(norms[0][2].dtype) if norms else F32
+    _check(fn(ctypes.byref(p), _stream()), "rmsnorm")
 
 
 def rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, *, num_heads: int, num_kv_heads: int, head_dim: int,
@@ -1532,23 +1573,24 @@ class _LatentParams(ctypes.Structure):
         ("part", _c_void), ("split_keys", _c_int), ("num_splits", _c_int),
         ("stage", _c_int), ("padded_tokens", _c_int), ("a_heads", _c_void), ("qa_heads", _c_void), ("q_rot", _c_void),
         ("l_heads", _c_void), ("o_heads", _c_void), ("tile_group", _c_void),
-        ("window", _c_int), ("pairing", _c_int),
+        ("window", _c_int), ("pairing", _c_int), ("sink", _c_void), ("q", _c_void), ("q_width", ctypes.c_longlong),
+        ("cq_off", _c_int), ("q_rank", _c_int), ("cq_norm_weight", _c_void), ("cq", _c_void),
     ]
 
 
 @functools.lru_cache(maxsize=4096)
-def latent_plan(tokens: int, heads: int, max_keys: int, sm_count: int):
+def latent_plan(tokens: int, heads: int, max_keys: int, sm_count: int, window: int = 0):
     """How the tensor-core fold over the latents cuts a step: (tokens per tile, heads per tile,
-    keys per split, splits)."""
-    fn = _function("latent", "vipera_latent_plan", [_c_int] * 4 + [ctypes.POINTER(_c_int)])
+    keys per split, splits).  With a window the splits cover the window only."""
+    fn = _function("latent", "vipera_latent_plan", [_c_int] * 5 + [ctypes.POINTER(_c_int)])
     plan = (_c_int * 4)()
-    _check(fn(int(tokens), int(heads), int(max_keys), int(sm_count), plan), "latent_plan", kernels=0)
+    _check(fn(int(tokens), int(heads), int(max_keys), int(window or 0), int(sm_count), plan), "latent_plan", kernels=0)
     return tuple(plan)
 
 
-def latent_part_floats(tokens: int, heads: int, rank: int, max_keys: int, sm_count: int) -> int:
+def latent_part_floats(tokens: int, heads: int, rank: int, max_keys: int, sm_count: int, window: int = 0) -> int:
     """Floats of scratch the fold's splits need for a step (0 when it runs without splits)."""
-    splits = latent_plan(tokens, heads, max_keys, sm_count)[3]
+    splits = latent_plan(tokens, heads, max_keys, sm_count, window)[3]
     return splits * tokens * heads * (rank + 2) if splits > 1 else 0
 
 
@@ -1558,7 +1600,8 @@ def latent_attention(proj: torch.Tensor, *, q_off: int, g_off: int, kv_off: int,
                      v_pool: torch.Tensor, qa: torch.Tensor, latent_out: torch.Tensor, out: torch.Tensor, heads: int,
                      head_dim: int, rot_dim: int, value_dim: int, scale: float, max_keys: int = 0,
                      part: Optional[torch.Tensor] = None, head_major: Optional[dict] = None, window: int = 0,
-                     pairing: int = ROPE_INTERLEAVED) -> None:
+                     pairing: int = ROPE_INTERLEAVED, sink: Optional[torch.Tensor] = None,
+                     q: Optional[torch.Tensor] = None) -> None:
     """Causal softmax attention whose keys and values are products of a cached latent.  ``proj``
     float32 [tokens, width] holds q (head by head [head_dim | rot_dim]) at column ``q_off``, the
     output gate's pre-activation at ``g_off`` (negative: no gate) and the down projection
@@ -1577,7 +1620,10 @@ def latent_attention(proj: torch.Tensor, *, q_off: int, g_off: int, kv_off: int,
     rot_dim]), ``l_heads`` (bfloat16 [heads * padded, rank]), ``o_heads`` (float32 [heads * padded,
     value_dim]) and ``tile_group`` (int32 [heads * padded / 128]).  ``window`` > 0: a query at position
     p sees keys p - window + 1 .. p.  ``pairing``: which values of the rotated part turn together,
-    ROPE_INTERLEAVED (2i, 2i + 1) or ROPE_NEOX (i, i + rot_dim / 2)."""
+    ROPE_INTERLEAVED (2i, 2i + 1) or ROPE_NEOX (i, i + rot_dim / 2).  ``sink`` (float32 [heads]):
+    exp(sink_h) joins the softmax's denominator.  ``q`` (float32 [tokens, heads * (head_dim +
+    rot_dim)]): the queries, where they are no columns of ``proj`` (``q_off`` is then a column of q);
+    the cache is then written ahead of this call, by latent_store, and ``kv_off`` is negative."""
     fn = _function("latent", "vipera_latent_attention", [ctypes.POINTER(_LatentParams), _c_int, _c_void])
     _check_struct("latent", "vipera_latent_params_size", _LatentParams)
     tokens = proj.shape[0]
@@ -1599,6 +1645,13 @@ def latent_attention(proj: torch.Tensor, *, q_off: int, g_off: int, kv_off: int,
     p = _LatentParams()
     p.proj, p.proj_width = _gpu(proj, "proj", torch.float32), proj.shape[1]
     p.q_off, p.g_off, p.kv_off = int(q_off), int(g_off), int(kv_off)
+    if sink is not None and sink.numel() != heads:
+        raise InvalidArgumentError("latent_attention: one sink per head")
+    p.sink = _opt(sink, "sink", torch.float32)
+    if q is not None:
+        if q.shape[0] != tokens or q.shape[1] < q_off + heads * (head_dim + rot_dim):
+            raise InvalidArgumentError("latent_attention: q must hold every head's values")
+        p.q, p.q_width = _gpu(q, "q", torch.float32), q.shape[1]
     p.up_k, p.up_v = _gpu(up_k, "up_k"), _gpu(up_v, "up_v")
     p.norm_weight = _opt(norm_weight, "norm_weight", torch.float32)
     p.positions = _gpu(positions, "positions", torch.int32)
@@ -1616,7 +1669,7 @@ def latent_attention(proj: torch.Tensor, *, q_off: int, g_off: int, kv_off: int,
     p.window, p.pairing = int(window or 0), 1 if pairing == ROPE_NEOX else 0
     p.part, p.split_keys, p.num_splits = None, 0, 1
     if part is not None and max_keys > 0:
-        _, _, split_keys, splits = latent_plan(tokens, heads, int(max_keys), sm_count(proj.device))
+        _, _, split_keys, splits = latent_plan(tokens, heads, int(max_keys), sm_count(proj.device), p.window)
         if splits > 1:
             if part.numel() < splits * tokens * heads * (rank + 2):
                 raise InvalidArgumentError("latent_attention: the scratch of the splits is too small")
@@ -1645,6 +1698,43 @@ def latent_attention(proj: torch.Tensor, *, q_off: int, g_off: int, kv_off: int,
         _check(fn(ctypes.byref(p), code, _stream()), "attention")
         return
     _check(fn(ctypes.byref(p), dtype_code(k_pool.dtype), _stream()), "attention", kernels=4 if kv_off >= 0 else 3)
+
+
+def latent_store(proj: torch.Tensor, *, kv_off: int, norm_weight: Optional[torch.Tensor], eps: float,
+                 positions: torch.Tensor, token_entry: torch.Tensor, block_table: torch.Tensor, cos: torch.Tensor,
+                 sin: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, rot_dim: int,
+                 pairing: int = ROPE_INTERLEAVED, cq_off: int = -1, cq_norm_weight: Optional[torch.Tensor] = None,
+                 cq: Optional[torch.Tensor] = None) -> None:
+    """Ahead of latent_attention where the queries come through a latent of their own: the step's
+    normed latents and rotated key parts (columns ``kv_off`` of ``proj``; negative: none) into their
+    pages, and the query latents (columns ``cq_off``, ``cq.shape[1]`` of them), RMS-normed with
+    ``cq_norm_weight``, into ``cq`` in the pools' type."""
+    fn = _function("latent", "vipera_latent_attention", [ctypes.POINTER(_LatentParams), _c_int, _c_void])
+    _check_struct("latent", "vipera_latent_params_size", _LatentParams)
+    page_size, rank = k_pool.shape[1], k_pool.shape[3]
+    if tuple(k_pool.shape[1:]) != (page_size, 1, rank) or tuple(v_pool.shape[1:]) != (page_size, 1, rot_dim) or \
+            k_pool.dtype != v_pool.dtype or tuple(cos.shape[1:]) != (rot_dim // 2,) or cos.shape != sin.shape:
+        raise InvalidArgumentError("latent_store: the pools or the cos/sin tables have the wrong shape")
+    if kv_off >= 0 and (norm_weight is None or norm_weight.numel() != rank or kv_off + rank + rot_dim > proj.shape[1]):
+        raise InvalidArgumentError("latent_store: the latent's columns or its norm weight do not match")
+    p = _LatentParams()
+    p.proj, p.proj_width, p.kv_off, p.g_off = _gpu(proj, "proj", torch.float32), proj.shape[1], int(kv_off), -1
+    p.norm_weight = _opt(norm_weight, "norm_weight", torch.float32)
+    p.positions = _gpu(positions, "positions", torch.int32)
+    p.token_entry = _gpu(token_entry, "token_entry", torch.int32)
+    p.block_table = _gpu(block_table, "block_table", torch.int32)
+    p.cos_table, p.sin_table = _gpu(cos, "cos", torch.float32), _gpu(sin, "sin", torch.float32)
+    p.k_pool, p.v_pool = _gpu(k_pool, "k_pool"), _gpu(v_pool, "v_pool")
+    p.num_tokens, p.heads, p.d, p.rot, p.dv, p.rank = int(proj.shape[0]), 1, 1, int(rot_dim), 1, int(rank)
+    p.table_width, p.page_size, p.eps = int(block_table.shape[1]), int(page_size), float(eps)
+    p.pairing, p.num_splits, p.stage = (1 if pairing == ROPE_NEOX else 0), 1, 4
+    if cq is not None:
+        if cq.shape[0] != proj.shape[0] or cq.dtype != k_pool.dtype or cq_norm_weight is None or \
+                cq_norm_weight.numel() != cq.shape[1] or not 0 <= cq_off <= proj.shape[1] - cq.shape[1]:
+            raise InvalidArgumentError("latent_store: the query latent's columns, norm weight or output do not match")
+        p.cq_off, p.q_rank = int(cq_off), int(cq.shape[1])
+        p.cq_norm_weight, p.cq = _gpu(cq_norm_weight, "cq_norm_weight", torch.float32), _gpu(cq, "cq")
+    _check(fn(ctypes.byref(p), dtype_code(k_pool.dtype), _stream()), "attention")
 
 
 # ----------------------------------------------------------------------------------------
@@ -1712,10 +1802,11 @@ class _MoeParams(ctypes.Structure):
         ("tile_expert", _c_void), ("act", _c_void), ("rows", _c_void), ("xs", _c_void), ("ys", _c_void),
         ("num_tokens", _c_int), ("hidden", _c_int), ("ff", _c_int), ("experts", _c_int), ("top", _c_int),
         ("groups", _c_int), ("keep", _c_int), ("group_top", _c_int), ("max_tiles", _c_int),
-        ("softmax_scores", _c_int), ("renormalize", _c_int), ("activation", _c_int),
+        ("scores", _c_int), ("renormalize", _c_int), ("activation", _c_int),
         ("gate_group", _c_int), ("tile_rows", _c_int), ("padded", _c_int),
         ("correction", _c_void), ("identity", _c_int), ("always", _c_int), ("slots", _c_int), ("gated", _c_int),
         ("route_scale", _c_float), ("renorm_eps", _c_float),
+        ("always_gate", _c_int), ("unit_limit", _c_void), ("unit_slope", _c_float),
     ]
 
 
@@ -1750,12 +1841,17 @@ def moe_scratch_words(tokens: int, top: int, experts: int) -> int:
 
 
 def gemm_tc_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, *, epilogue: int, out: torch.Tensor,
-                    activation: int = ACT_SILU, what: str = "gemm_tc") -> None:
+                    activation: int = ACT_SILU, unit_limit: Optional[torch.Tensor] = None, unit_slope: float = 0.0,
+                    what: str = "gemm_tc") -> None:
     """a[M, K] (M a multiple of 128) times one of the matrices w[G, N, K], transposed: rows 128 i ..
     128 i + 127 use matrix tile_group[i] (int32, written on the device ahead of this call).
-    Endings: plain store, or the gated unit over interleaved gate and up rows."""
+    Endings: plain store, or the gated unit over interleaved gate and up rows (with ACT_CLAMPED each
+    group's unit has the bound ``unit_limit[group]``, float32, and ``unit_slope``)."""
     fn = _function("gemm_tc", "vipera_gemm_tc_grouped",
-                   [_c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int, _c_int, _c_void, _c_void])
+                   [_c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_void, _c_int, _c_void, _c_int, _c_int, _c_void,
+                    _c_float, _c_void, _c_void])
+    if activation == ACT_CLAMPED and (unit_limit is None or unit_limit.numel() != w.shape[0]):
+        raise InvalidArgumentError("gemm_tc_grouped: one bound per group")
     m, k = a.shape
     groups, n = w.shape[0], w.shape[1]
     if w.shape[2] != k or m % 128 or tile_group.numel() < m // 128 or k % 8:
@@ -1766,6 +1862,7 @@ def gemm_tc_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, 
     state = _tc_buffers(a.device, 0)
     _check(fn(_gpu(a, "a", torch.bfloat16), _gpu(w, "w", torch.bfloat16), m, n, k, groups,
               _gpu(tile_group, "tile_group", torch.int32), epilogue, _gpu(out, "out"), dtype_code(out.dtype), int(activation),
+              _opt(unit_limit, "unit_limit", torch.float32), float(unit_slope),
               state["status"].data_ptr(), _stream()), what)
 
 
@@ -1774,7 +1871,8 @@ def moe(h: torch.Tensor, *, router: torch.Tensor, gate_up: torch.Tensor, down: t
         chosen: torch.Tensor, weight: torch.Tensor, scratch: torch.Tensor, act: torch.Tensor, rows: torch.Tensor,
         xs: Optional[torch.Tensor] = None, ys: Optional[torch.Tensor] = None, gated: bool = True,
         correction: Optional[torch.Tensor] = None, identity: int = 0, always: int = 0, route_scale: float = 1.0,
-        renorm_eps: float = 0.0) -> None:
+        renorm_eps: float = 0.0, logit_scores: bool = False, always_gate: bool = False,
+        unit_limit: Optional[torch.Tensor] = None, unit_slope: float = 0.0) -> None:
     """A mixture of gated units over a step.  ``h`` [tokens, hidden]; ``router`` float32 [experts,
     hidden]; ``gate_up`` [experts, 2 ff, hidden] (``gate_group`` gate rows, then the up rows of the
     same features, and so on) and ``down`` [experts, hidden, ff] in h's type.  ``chosen`` int32 and
@@ -1791,12 +1889,19 @@ def moe(h: torch.Tensor, *, router: torch.Tensor, gate_up: torch.Tensor, down: t
     token uses with weight 1; ``top`` stays the router's count, and ``chosen``, ``weight`` and ``rows``
     hold ``top + always`` places per token, sized by the caller with moe_capacity(tokens, top + always,
     matrices) and so on.  ``renormalize`` divides the weights by their sum + ``renorm_eps``;
-    ``route_scale`` multiplies them."""
+    ``route_scale`` multiplies them.  ``logit_scores``: the scores are the logits themselves, and the
+    weights the softmax over the chosen ones.  ``always_gate``: ``router`` has one row more, and the
+    always-used units' weight is the sigmoid of its product with h.  Activation ACT_CLAMPED: gated units
+    with the bounds ``unit_limit`` (float32, one per unit with matrices) and ``unit_slope``."""
     fn = _function("moe", "vipera_moe", [ctypes.POINTER(_MoeParams), _c_int, _c_void])
     _check_struct("moe", "vipera_moe_params_size", _MoeParams)
     tokens, hidden = h.shape
     matrices, ff = gate_up.shape[0], gate_up.shape[1] // (2 if gated else 1)
-    outputs, identity, always = router.shape[0], int(identity), int(always)
+    outputs, identity, always = router.shape[0] - int(bool(always_gate)), int(identity), int(always)
+    if activation == ACT_CLAMPED and (not gated or unit_limit is None or unit_limit.numel() != matrices):
+        raise InvalidArgumentError("moe: the bounded activation needs gated units and one bound per unit")
+    if always_gate and not always:
+        raise InvalidArgumentError("moe: a gate of the always-used units without such units")
     if outputs - identity + always != matrices or identity < 0 or always < 0 or router.shape[1] != hidden or \
             tuple(gate_up.shape) != (matrices, (2 if gated else 1) * ff, hidden) or \
             tuple(down.shape) != (matrices, hidden, ff) or gate_up.dtype != h.dtype or down.dtype != h.dtype:
@@ -1830,7 +1935,10 @@ def moe(h: torch.Tensor, *, router: torch.Tensor, gate_up: torch.Tensor, down: t
     p.identity, p.always, p.slots, p.gated = identity, always, top, int(bool(gated))
     p.route_scale, p.renorm_eps = float(route_scale), float(renorm_eps)
     p.groups, p.keep, p.group_top, p.max_tiles = int(groups), int(keep), int(group_top), int(tiles)
-    p.softmax_scores, p.renormalize, p.activation = int(bool(softmax_scores)), int(bool(renormalize)), int(activation)
+    p.scores = 2 if logit_scores else int(bool(softmax_scores))
+    p.renormalize, p.activation = int(bool(renormalize)), int(activation)
+    p.always_gate, p.unit_slope = int(bool(always_gate)), float(unit_slope)
+    p.unit_limit = _opt(unit_limit, "unit_limit", torch.float32)
     p.gate_group, p.tile_rows, p.padded = int(gate_group), int(tile_rows), int(padded)
     if not padded:
         _check(fn(ctypes.byref(p), dtype_code(h.dtype), _stream()), "moe", kernels=4)
@@ -1844,7 +1952,8 @@ def moe(h: torch.Tensor, *, router: torch.Tensor, gate_up: torch.Tensor, down: t
     act_rows = act.view(-1)[:capacity * ff].view(capacity, ff)
     ys_rows = ys.view(-1)[:capacity * hidden].view(capacity, hidden)
     gemm_tc_grouped(xs_rows, gate_up, tile_expert, epilogue=EPI_GATED if gated else EPI_STORE, out=act_rows,
-                    activation=activation, what="moe")
+                    activation=activation, unit_limit=unit_limit if activation == ACT_CLAMPED else None,
+                    unit_slope=unit_slope, what="moe")
     gemm_tc_grouped(act_rows, down, tile_expert, epilogue=EPI_STORE, out=ys_rows, what="moe")
     scatter = _function("moe", "vipera_moe_scatter", [ctypes.POINTER(_MoeParams), _c_void])
     _check(scatter(ctypes.byref(p), _stream()), "moe")

@@ -13,6 +13,9 @@ Mixer           ``cache_request()`` says what the mixer keeps between steps (pag
                 values, a fixed-size state, or nothing); ``forward(ctx, h, residual, cache,
                 writes_cache)`` adds the mixer's output into ``residual`` in place.
 FeedForward     ``forward(ctx, h, residual)`` adds its output into ``residual`` in place.
+                (A mixer or feed-forward that sets ``leaves_rows`` may be handed None as its
+                ``residual``: it then leaves its output and returns (rows [tokens, parts * hidden]
+                float32, parts), the output being the sum of a token's parts in their order.)
 Block           ``forward(ctx, residual, cache, writes_cache)`` arranges the four.
 
 The reference's seam between runtime and backend is the same in spirit: the backend turns
@@ -182,6 +185,7 @@ class StepContext:
     dtype: torch.dtype          # activation dtype of the run
     workspace: Workspace
     logits_all_rows: bool = False  # the wanted rows are all the step's tokens, in order
+    pending: Optional[Any] = None  # branches that have yet to join the stream (see block.PendingJoin)
     extras: Dict[str, Any] = field(default_factory=dict)
 
 

@@ -34,6 +34,7 @@ class Block:
 
     roles: Dict[str, Registry] = {}
     cache_role = "mixer"
+    takes_pending = False   # True: forward() adds what the layer before left pending itself
 
     def __init__(self, layer_spec, tensors, dtype, device):
         self.spec = layer_spec
@@ -323,7 +324,125 @@ class SandwichBlock(Block):
             self._join(ctx, "ffn", h, rows[0], rows[1], residual)
 
 
+class PendingJoin:
+    """Branches of a layer that have been computed and not yet added to the stream: ``(rows, parts,
+    scale)`` each, ``x += scale * sum of the parts``.  Whoever reads the stream next adds them on the way:
+    a ``parallel`` layer and the model's last norm in the kernel that computes their norms, anything else
+    after ``settle``."""
+
+    def __init__(self, branches):
+        self.branches = list(branches)
+
+    @staticmethod
+    def settle(ctx, residual) -> None:
+        """Add what is pending, if anything is."""
+        pending, ctx.pending = ctx.pending, None
+        if pending is not None:
+            ops.join_norms(residual, pending.branches)
+
+    @staticmethod
+    def takes(norm) -> bool:
+        """Whether the joining kernel computes this norm."""
+        return getattr(norm, "fused_kind", None) == "rmsnorm" and getattr(norm, "weight", None) is not None
+
+    @staticmethod
+    def normed(ctx, residual, norms, names, rows=None):
+        """The norms of the stream with what is pending added to it, one tensor each.  With ``rows`` only
+        those rows are read and the stream is left as it is (for its last reader)."""
+        count = residual.shape[0] if rows is None else rows.numel()
+        outs = [ctx.workspace.get(name, (count, residual.shape[1]), ctx.dtype) for name in names]
+        if all(PendingJoin.takes(norm) for norm in norms):
+            pending, ctx.pending = ctx.pending, None
+            ops.join_norms(residual, pending.branches if pending is not None else (),
+                           [(norm.weight, norm.eps, out) for norm, out in zip(norms, outs)], rows)
+        else:
+            PendingJoin.settle(ctx, residual)
+            for norm, out in zip(norms, outs):
+                norm.forward(ctx, residual, out, rows=rows)
+        return outs
+
+
+class ParallelBlock(Block):
+    """Mixer and feed-forward side by side: both read the same stream, each through a norm of its own,
+    and their outputs join it together,
+
+        x += s1 * mixer(N1(x)) + s2 * ff(N2(x))
+
+    (the second term only where the layer has a feed-forward).  ``params``: ``hidden_size`` and
+    ``layer_scale`` (true: tensors ``<layer>.<mixer_scale>.weight`` and ``<layer>.<ffn_scale>.weight``
+    [hidden], the s above; false: 1).  The branches are left for the next reader of the stream to add
+    (``PendingJoin``): one kernel adds a layer's branches, with their scales and the sum over a token's
+    expert rows, and computes both norms of the next layer."""
+
+    roles = {"mixer_norm": NORMS, "mixer": MIXERS}
+    optional_roles = {"ffn_norm": NORMS, "ffn": FEED_FORWARDS}
+    takes_pending = True
+
+    def __init__(self, layer_spec, tensors, dtype, device):
+        self.roles = self._roles_of(layer_spec)
+        super().__init__(layer_spec, tensors, dtype, device)
+        self.hidden = int(layer_spec.params["hidden_size"])
+        self.sides = self._sides(layer_spec)
+        self.scales = {side: None for side in self.sides}
+        if layer_spec.params.get("layer_scale", False):
+            for side in self.sides:
+                scale = tensors[f"{layer_spec.part_prefix(side + '_scale')}.weight"]
+                self.scales[side] = scale.to(device=device, dtype=torch.float32).contiguous()
+
+    @staticmethod
+    def _sides(layer_spec):
+        return ("mixer", "ffn") if "ffn" in layer_spec.parts else ("mixer",)
+
+    @classmethod
+    def _roles_of(cls, layer_spec):
+        roles = dict(cls.roles)
+        if "ffn" in layer_spec.parts:
+            roles.update(cls.optional_roles)
+        return roles
+
+    @classmethod
+    def schema(cls, layer_spec):
+        schema = {}
+        for role, registry in cls._roles_of(layer_spec).items():
+            part_spec = cls._role_spec(layer_spec, role)
+            schema.update(registry.find(part_spec.kind).schema(part_spec.params, layer_spec.part_prefix(role)))
+        if layer_spec.params.get("layer_scale", False):
+            for side in cls._sides(layer_spec):
+                schema[f"{layer_spec.part_prefix(side + '_scale')}.weight"] = TensorSpec(
+                    (int(layer_spec.params["hidden_size"]),), init="layer_scale", store="float32")
+        return schema
+
+    @classmethod
+    def workspace_bytes(cls, layer_spec, tokens, element_bytes):
+        # both branches' rows and both norms' outputs
+        total = 2 * tokens * int(layer_spec.params["hidden_size"]) * (4 + element_bytes)
+        for role, registry in cls._roles_of(layer_spec).items():
+            part_spec = cls._role_spec(layer_spec, role)
+            total += registry.find(part_spec.kind).workspace_bytes(part_spec.params, tokens, element_bytes)
+        return total
+
+    def _branch(self, ctx, side, run):
+        """What one side adds to the stream.  A part that cannot leave rows adds into a cleared buffer."""
+        part = self._parts[side]
+        if getattr(part, "leaves_rows", False):
+            rows, parts = run(part, None)
+        else:
+            rows, parts = ctx.workspace.get(f"block.{side}_rows", (ctx.num_tokens, self.hidden), torch.float32), 1
+            rows.zero_()
+            run(part, rows)
+        return rows, parts, self.scales[side]
+
+    def forward(self, ctx, residual, cache, writes_cache):
+        norms = [self._parts[f"{side}_norm"] for side in self.sides]
+        inputs = PendingJoin.normed(ctx, residual, norms, ["block.h", "block.h2"][:len(norms)])
+        branches = [self._branch(ctx, "mixer", lambda part, into: part.forward(ctx, inputs[0], into, cache, writes_cache))]
+        if "ffn" in self._parts:
+            branches.append(self._branch(ctx, "ffn", lambda part, into: part.forward(ctx, inputs[1], into)))
+        ctx.pending = PendingJoin(branches)
+
+
 BLOCKS.register("prenorm", PreNormBlock)
+BLOCKS.register("parallel", ParallelBlock)
 BLOCKS.register("sandwich", SandwichBlock)
 BLOCKS.register("outnorm_conv", OutNormConvBlock)
 BLOCKS.register("prenorm_mixer", PreNormMixerBlock)

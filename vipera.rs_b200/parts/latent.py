@@ -4,7 +4,9 @@ From the mixer's input h: ``q = W_q h`` (head by head ``[d unrotated | r rotated
 ``W_dkv h = [c' | k_r']``; the latent ``c = rmsnorm(c') * w`` [rank] and the rotated key part
 ``k_r = rot(k_r')`` [r], shared by all heads, are all a token leaves in the cache.  Head h's key
 is ``[U_h c | k_r]`` and its value ``V_h c``; the score is ``scale * (q_d . U_h c + rot(q_r) . k_r)``,
-the mask causal, the softmax plain.  The concatenated heads are multiplied by ``sigmoid(W_g h)``
+the mask causal.  Options: the queries come through a normed latent of their own, ``q = W_uq
+rmsnorm(W_dq h)`` (``q_rank``); a window; a softmax whose denominator also holds ``exp(sink_h)``, a
+learned number per head that stands for no token (``sink``).  The concatenated heads are multiplied by ``sigmoid(W_g h)``
 (where the mixer has an output gate) and sent through the output matrix, which adds into the stream
 the mixer is handed.
 
@@ -38,23 +40,34 @@ class LatentAttention(Mixer):
     values per head; the key's are shared), value_dim, kv_rank, softmax_scale, norm_eps, position (a
     PartSpec of a rotary encoding over rot_dim values: interleaved pairs or halves) and, optionally,
     ``own_cache`` (default true), ``output_gate`` (default false), ``window`` (a query at position p
-    sees keys p - window + 1 .. p; pages the window has left are given back).  Tensors under ``<prefix>``: q [heads * (head_dim +
-    rot_dim), hidden], dkv [kv_rank + rot_dim, hidden] and dkv.norm [kv_rank] (with a cache of its
-    own), uk [heads * head_dim, kv_rank], uv [heads * value_dim, kv_rank], g [heads * value_dim,
-    hidden] (with a gate), o [hidden, heads * value_dim]."""
+    sees keys p - window + 1 .. p; pages the window has left are given back), ``q_rank`` (the size of a
+    latent the queries come through), ``sink`` (``"learned"``: a number per head joins the softmax's
+    denominator).  Tensors under ``<prefix>``: q [heads * (head_dim + rot_dim), hidden] (with a query
+    latent instead dq [q_rank, hidden], dq.norm [q_rank] and uq [heads * (head_dim + rot_dim), q_rank]),
+    dkv [kv_rank + rot_dim, hidden] and dkv.norm [kv_rank] (with a cache of its own), uk [heads *
+    head_dim, kv_rank], uv [heads * value_dim, kv_rank], sink [heads], g [heads * value_dim, hidden]
+    (with a gate), o [hidden, heads * value_dim]."""
 
     kernels = ("latent",)
+    leaves_rows = True   # forward(ctx, h, None, ...) returns (rows [tokens, hidden] float32, 1)
 
     @classmethod
     def schema(cls, params, prefix):
         hidden, heads = params["hidden_size"], params["num_heads"]
         d, r, dv, rank = params["head_dim"], params["rot_dim"], params["value_dim"], params["kv_rank"]
-        schema = {
-            f"{prefix}.q.weight": TensorSpec((heads * (d + r), hidden)),
+        q_rank = int(params.get("q_rank") or 0)
+        schema = {f"{prefix}.q.weight": TensorSpec((heads * (d + r), hidden))} if not q_rank else {
+            f"{prefix}.dq.weight": TensorSpec((q_rank, hidden)),
+            f"{prefix}.dq.norm.weight": TensorSpec((q_rank,), init="norm", store="float32"),
+            f"{prefix}.uq.weight": TensorSpec((heads * (d + r), q_rank)),
+        }
+        if params.get("sink"):
+            schema[f"{prefix}.sink.weight"] = TensorSpec((heads,), init="sink", store="float32")
+        schema.update({
             f"{prefix}.uk.weight": TensorSpec((heads * d, rank)),
             f"{prefix}.uv.weight": TensorSpec((heads * dv, rank)),
             f"{prefix}.o.weight": TensorSpec((hidden, heads * dv)),
-        }
+        })
         if params.get("own_cache", True):
             schema[f"{prefix}.dkv.weight"] = TensorSpec((rank + r, hidden))
             schema[f"{prefix}.dkv.norm.weight"] = TensorSpec((rank,), init="norm")
@@ -74,12 +87,21 @@ class LatentAttention(Mixer):
         if self.rank > ops.LATENT_MAX_RANK or self.rot > ops.LATENT_MAX_ROT or self.rot % 2:
             raise UnsupportedError(f"{prefix}: latent attention takes a rank up to {ops.LATENT_MAX_RANK} and an even "
                                    f"rotated part up to {ops.LATENT_MAX_ROT}")
-        # one product for everything that reads h: q, the gate's pre-activation, the down projection
-        names = ["q"] + (["g"] if self.gated else []) + (["dkv"] if self.own_cache else [])
+        self.q_rank = int(params.get("q_rank") or 0)
+        if params.get("sink") not in (None, "learned"):
+            raise UnsupportedError(f"{prefix}: a sink of latent attention is learned, not {params['sink']!r}")
+        # one product for everything that reads h: q (or its latent), the gate's pre-activation, the down projection
+        names = ["dq" if self.q_rank else "q"] + (["g"] if self.gated else []) + (["dkv"] if self.own_cache else [])
         rows = [tensors[f"{prefix}.{name}.weight"] for name in names]
         starts = {name: sum(r.shape[0] for r in rows[:i]) for i, name in enumerate(names)}
-        self.q_off, self.g_off, self.kv_off = starts["q"], starts.get("g", -1), starts.get("dkv", -1)
+        self.q_off, self.g_off, self.kv_off = starts[names[0]], starts.get("g", -1), starts.get("dkv", -1)
         self.proj = Linear(torch.cat(rows, dim=0), dtype, device)
+        self.up_q = self.q_norm = self.sink = None
+        if self.q_rank:
+            self.up_q = Linear(tensors[f"{prefix}.uq.weight"], dtype, device)
+            self.q_norm = tensors[f"{prefix}.dq.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
+        if params.get("sink"):
+            self.sink = tensors[f"{prefix}.sink.weight"].to(device=device, dtype=torch.float32).contiguous()
         self.up_k = tensors[f"{prefix}.uk.weight"].to(device=device, dtype=dtype).contiguous()
         # each head's value matrix transposed, [heads, rank, value_dim]: neighbouring threads read neighbouring values
         self.up_v = tensors[f"{prefix}.uv.weight"].to(device=device, dtype=dtype).view(
@@ -104,7 +126,8 @@ class LatentAttention(Mixer):
 
     def kernel_families(self):
         grouped = ("gemm_tc",) if self.head_major else ()
-        return tuple(dict.fromkeys(("latent",) + grouped + self.proj.kernel_families() + self.out.kernel_families()))
+        up_q = self.up_q.kernel_families() if self.up_q is not None else ()
+        return tuple(dict.fromkeys(("latent",) + grouped + self.proj.kernel_families() + up_q + self.out.kernel_families()))
 
     def prepare(self, max_positions: int) -> None:
         self.position.prepare(max_positions)
@@ -116,7 +139,7 @@ class LatentAttention(Mixer):
     @classmethod
     def workspace_bytes(cls, params, tokens, element_bytes):
         heads, rank, r = params["num_heads"], params["kv_rank"], params["rot_dim"]
-        width = heads * (params["head_dim"] + r + params["value_dim"]) + rank + r
+        width = heads * (params["head_dim"] + r + params["value_dim"]) + rank + r + 2 * int(params.get("q_rank") or 0)
         # (the splits of a step of few tokens: at most some 600 blocks of 16 rows more than the step's own)
         padded = tokens + 127
         head_major = heads * padded * (params["head_dim"] * 2 + rank * 6 + params["value_dim"] * 4) + tokens * heads * r * 4 + 4096
@@ -134,8 +157,7 @@ class LatentAttention(Mixer):
         mixed = ws.get("latent.out", (count, self.heads * self.vdim), ctx.dtype)
         cos, sin = self.position.tables()
         max_keys = max(int(ctx.max_kv_len), 1)
-        # (with a window the splits past it see no key and leave at once; the combine skips them)
-        floats = ops.latent_part_floats(count, self.heads, self.rank, max_keys, ops.sm_count(h.device)) if ctx.dtype == torch.bfloat16 else 0
+        floats = ops.latent_part_floats(count, self.heads, self.rank, max_keys, ops.sm_count(h.device), self.window) if ctx.dtype == torch.bfloat16 else 0
         part = ws.get("latent.part", (floats,), torch.float32) if floats else None
         head_major = None
         if self.head_major and count >= HEAD_MAJOR_FROM:
@@ -149,13 +171,30 @@ class LatentAttention(Mixer):
                 "o_heads": ws.get("latent.o_heads", (self.heads * padded, self.vdim), torch.float32),
                 "tile_group": ws.get("latent.tile_group", (self.heads * padded // 128,), torch.int32),
             }
-        ops.latent_attention(proj, q_off=self.q_off, g_off=self.g_off, kv_off=self.kv_off, up_k=self.up_k, up_v=self.up_v,
+        q, q_off, kv_off = None, self.q_off, self.kv_off
+        if self.q_rank:
+            # the norm of the query latent shares a kernel with the cache write; its product follows
+            cq = ws.get("latent.cq", (count, self.q_rank), ctx.dtype)
+            ops.latent_store(proj, kv_off=kv_off, norm_weight=self.latent_norm, eps=self.norm_eps, positions=ctx.positions,
+                             token_entry=ctx.token_entry, block_table=ctx.block_tables[cache.group], cos=cos, sin=sin,
+                             k_pool=cache.k, v_pool=cache.v, rot_dim=self.rot, pairing=self.position.style,
+                             cq_off=self.q_off, cq_norm_weight=self.q_norm, cq=cq)
+            q = ws.get("latent.q", (count, self.up_q.out_features), torch.float32)
+            self.up_q(ctx, cq, epilogue=ops.EPI_STORE, out=q)
+            q_off, kv_off = 0, -1
+        ops.latent_attention(proj, q_off=q_off, g_off=self.g_off, kv_off=kv_off, up_k=self.up_k, up_v=self.up_v,
                              norm_weight=self.latent_norm, eps=self.norm_eps, positions=ctx.positions,
                              token_entry=ctx.token_entry, block_table=ctx.block_tables[cache.group], cos=cos, sin=sin,
                              k_pool=cache.k, v_pool=cache.v, qa=qa, latent_out=mixed_latent, out=mixed, heads=self.heads,
                              head_dim=self.dim, rot_dim=self.rot, value_dim=self.vdim, scale=self.scale, max_keys=max_keys,
-                             part=part, head_major=head_major, window=self.window, pairing=self.position.style)
+                             part=part, head_major=head_major, window=self.window, pairing=self.position.style,
+                             sink=self.sink, q=q)
+        if residual is None:
+            rows = ws.get("latent.rows", (count, self.hidden), torch.float32)
+            self.out(ctx, mixed, epilogue=ops.EPI_STORE, out=rows)
+            return rows, 1
         self.out(ctx, mixed, epilogue=ops.EPI_RESIDUAL, resid=residual)
+        return None
 
 
 MIXERS.register("latent_attention", LatentAttention)

@@ -57,6 +57,10 @@ class NormedInput:
         return (getattr(self.norm, "fused_kind", None) == "rmsnorm" and weight is not None
                 and weight.dtype == torch.float32)
 
+    def preset(self, tensor: torch.Tensor) -> None:
+        """The normalised rows, where something else has computed them."""
+        self._tensor = tensor
+
     def tensor(self) -> torch.Tensor:
         if self._tensor is None:
             out = self.ctx.workspace.get(self.name, (self.num_rows, self.residual.shape[1]), self.ctx.dtype)

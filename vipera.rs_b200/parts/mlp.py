@@ -25,6 +25,7 @@ class SwiGLU(FeedForward):
     projections then have one, ``<name>.bias``).  Registered as ``swiglu`` and ``gated_mlp``."""
 
     takes_lazy_input = True
+    leaves_rows = True   # forward(ctx, h, None) returns (rows [tokens, hidden] float32, 1)
 
     @staticmethod
     def _names(params):
@@ -89,7 +90,12 @@ class SwiGLU(FeedForward):
     def forward(self, ctx, h, residual):
         act = ctx.workspace.get("swiglu.act", (ctx.num_tokens, self.inter), ctx.dtype)
         self.gate_up(ctx, h, epilogue=ops.EPI_GATED, out=act, activation=self.activation)
+        if residual is None:
+            rows = ctx.workspace.get("swiglu.rows", (ctx.num_tokens, self.hidden), torch.float32)
+            self.down(ctx, act, epilogue=ops.EPI_STORE, out=rows)
+            return rows, 1
         self.down(ctx, act, epilogue=ops.EPI_RESIDUAL, resid=residual)
+        return None
 
 
 FEED_FORWARDS.register("swiglu", SwiGLU)

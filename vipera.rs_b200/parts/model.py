@@ -17,6 +17,7 @@ from ..errors import InternalError, InvalidArgumentError
 from ..kernels import ops
 from ..weights import Schema, TensorSpec, WeightSource, check_source, to_run_dtype
 from .base import StepContext
+from .block import PendingJoin
 from .linear import Linear, NormedInput
 
 
@@ -129,12 +130,18 @@ class DecoderModel:
         if self.embedding_norm is not None:
             # in place: the normed rows are the stream the first layer reads, in 32-bit
             self.embedding_norm.forward(ctx, residual, residual)
+        ctx.pending = None
         for entry in self.spec.schedule:
+            if not self.blocks[entry.layer].takes_pending:
+                PendingJoin.settle(ctx, residual)
             self.blocks[entry.layer].forward(ctx, residual, caches.get(entry.cache), entry.writes_cache)
         if ctx.num_logit_rows == 0:
             return None
         h = NormedInput(ctx, self.final_norm, residual, rows=ctx.logit_rows, num_rows=ctx.num_logit_rows,
                         name="model.final")
+        if ctx.pending is not None:
+            # the stream's last reader: its branches join on the way into the final norm
+            h.preset(PendingJoin.normed(ctx, residual, [self.final_norm], ["model.final"], rows=ctx.logit_rows)[0])
         logits = ws.get("model.logits", (ctx.num_logit_rows, self.spec.vocab_size), torch.float32)
         self.head(ctx, h, epilogue=ops.EPI_STORE, out=logits)
         if self.spec.logit_scale != 1.0:

@@ -23,7 +23,11 @@ which return the token's own row times their weight.  ``renorm_eps`` joins the s
 divided by, ``route_scale`` multiplies them.  A shared unit of the same form (``shared_size``, its
 inner size) that every token uses: since ``D act(U h)`` is a sum over the inner features, it is cut
 into pieces of the experts' inner size (the last filled up with zero features) that ride along as
-further units with weight 1, through the same tiles and products.
+further units with weight 1 (or, with ``shared_gate``, the sigmoid of one more row of the router times
+h), through the same tiles and products.  ``score`` = ``logit``: the choice is by the logits, the weights
+are the softmax over the chosen logits.  ``activation`` = ``clamped``: with g = G h bounded above by the
+unit's limit and u = U h held within it on both sides, ``D (g sigmoid(slope g) (u + 1))``; the shared
+unit has a limit of its own, and a feature filled up with zeros gives 0.
 """
 from __future__ import annotations
 
@@ -39,8 +43,10 @@ from .base import FeedForward
 class MixtureOfExperts(FeedForward):
     """params: hidden_size, intermediate_size (of one expert), experts, top and, optionally,
     ``groups`` (default 1), ``keep_groups`` (default: all), ``group_score_top`` (1 or 2, default 2),
-    ``score`` (``sigmoid``, the default, or ``softmax``), ``renormalize`` (default false),
-    ``activation`` (``silu`` or ``gelu_tanh``; without a gate also ``relu2``), ``projection_names``
+    ``score`` (``sigmoid``, the default, ``softmax`` or ``logit``), ``renormalize`` (default false),
+    ``activation`` (``silu``, ``gelu_tanh`` or ``clamped``, the latter with ``limit``, ``slope`` and
+    ``shared_limit``; without a gate silu, gelu_tanh or ``relu2``), ``shared_gate`` (true: tensor
+    ``<prefix>.shared.<shared_gate_name>.weight`` [1, hidden], the name ``gate`` by default), ``projection_names``
     (default gate, up, down), ``gated`` (default true; false: no gate matrices), ``identity`` (default 0:
     the last that many of the ``experts`` router outputs have no matrices), ``correction`` (true: tensor
     ``<prefix>.correction.weight`` [experts]), ``route_scale`` (default 1), ``renorm_eps`` (default 0),
@@ -64,6 +70,8 @@ class MixtureOfExperts(FeedForward):
         schema = {f"{prefix}.router.weight": TensorSpec((experts, hidden), store="float32")}
         if params.get("correction", False):
             schema[f"{prefix}.correction.weight"] = TensorSpec((experts,), init="correction", store="float32")
+        if params.get("shared_size") and params.get("shared_gate", False):
+            schema[cls._shared_gate_tensor(params, prefix)] = TensorSpec((1, hidden), store="float32")
         units = [(f"e{k}", inter) for k in range(experts - int(params.get("identity") or 0))]
         if params.get("shared_size"):
             units.append(("shared", int(params["shared_size"])))
@@ -73,6 +81,10 @@ class MixtureOfExperts(FeedForward):
             schema[f"{prefix}.{unit}.{up}.weight"] = TensorSpec((size, hidden))
             schema[f"{prefix}.{unit}.{down}.weight"] = TensorSpec((hidden, size))
         return schema
+
+    @staticmethod
+    def _shared_gate_tensor(params, prefix):
+        return f"{prefix}.shared.{params.get('shared_gate_name', 'gate')}.weight"
 
     @staticmethod
     def _counts(params):
@@ -97,13 +109,13 @@ class MixtureOfExperts(FeedForward):
         self.keep = int(params.get("keep_groups") or self.groups)
         self.group_top = int(params.get("group_score_top", 2))
         score = str(params.get("score", "sigmoid"))
-        if score not in ("sigmoid", "softmax"):
-            raise UnsupportedError(f"{prefix}: router scores are sigmoid or softmax, not {score!r}")
-        self.softmax_scores = score == "softmax"
+        if score not in ("sigmoid", "softmax", "logit"):
+            raise UnsupportedError(f"{prefix}: router scores are sigmoid, softmax or logit, not {score!r}")
+        self.softmax_scores, self.logit_scores = score == "softmax", score == "logit"
         self.renormalize = bool(params.get("renormalize", False))
         self.gated = bool(params.get("gated", True))
         name = str(params.get("activation", "silu"))
-        known = ops.ACTIVATIONS if self.gated else ops.UNIT_ACTIVATIONS
+        known = ops.BOUNDED_ACTIVATIONS if self.gated else ops.UNIT_ACTIVATIONS
         if name not in known:
             raise UnsupportedError(f"activation {name!r}; the unit knows: " + ", ".join(sorted(known)))
         self.activation = known[name]
@@ -124,6 +136,16 @@ class MixtureOfExperts(FeedForward):
                                    f"cannot give a token {self.top} experts")
         gate, up, down = self._names(params)
         self.router = tensors[f"{prefix}.router.weight"].to(device=device, dtype=torch.float32).contiguous()
+        self.shared_gate = bool(self.always and params.get("shared_gate", False))
+        if self.shared_gate:
+            row = tensors[self._shared_gate_tensor(params, prefix)].to(device=device, dtype=torch.float32)
+            self.router = torch.cat([self.router, row.view(1, self.hidden)], dim=0).contiguous()
+        self.unit_limit, self.unit_slope = None, 0.0
+        if self.activation == ops.ACT_CLAMPED:
+            own, shared = float(params["limit"]), float(params.get("shared_limit", params["limit"]))
+            self.unit_slope = float(params["slope"])
+            self.unit_limit = torch.tensor([own] * (self.matrices - self.always) + [shared] * self.always,
+                                           dtype=torch.float32, device=device)
 
         def stacked(which, features_last=False):
             """The units' matrices [matrices, ...]: the experts', then the shared unit's cut into pieces of
@@ -171,7 +193,8 @@ class MixtureOfExperts(FeedForward):
                 groups=self.groups, keep=self.keep, group_top=self.group_top, softmax_scores=self.softmax_scores,
                 renormalize=self.renormalize, activation=self.activation, chosen=chosen, weight=weight, scratch=scratch,
                 act=act, rows=rows, xs=xs, ys=ys, gated=self.gated, correction=self.correction, identity=self.identity,
-                always=self.always, route_scale=self.route_scale, renorm_eps=self.renorm_eps)
+                always=self.always, route_scale=self.route_scale, renorm_eps=self.renorm_eps, logit_scores=self.logit_scores,
+                always_gate=self.shared_gate, unit_limit=self.unit_limit, unit_slope=self.unit_slope)
         if residual is None:
             return rows, self.slots
         ops.add_rows(rows, self.slots, residual)

@@ -14,7 +14,8 @@ from .base import Norm
 class RMSNorm(Norm):
     """params: ``size`` (width of a row), ``eps`` and, optionally, ``groups`` (the row is cut into
     that many equal consecutive parts and each part is divided by its own root mean square; default
-    1, the whole row).  Tensor: ``<prefix>.weight`` [size].  The grouped form may write its 32-bit
+    1, the whole row) and ``weight_offset`` (default 0; 1 where the stored weight is the gain's
+    distance from one).  Tensor: ``<prefix>.weight`` [size].  The grouped form may write its 32-bit
     input in place."""
 
     kernels = ("rowwise",)
@@ -22,7 +23,8 @@ class RMSNorm(Norm):
 
     @classmethod
     def schema(cls, params, prefix):
-        return {f"{prefix}.weight": TensorSpec((params["size"],), init="norm", store="float32")}
+        init = "norm" if not params.get("weight_offset") else "centred_norm"
+        return {f"{prefix}.weight": TensorSpec((params["size"],), init=init, store="float32")}
 
     def __init__(self, params, prefix, tensors, dtype, device):
         super().__init__(params, prefix, tensors, dtype, device)
@@ -30,6 +32,8 @@ class RMSNorm(Norm):
         self.eps = float(params["eps"])
         # The weight is used in 32-bit whatever it was stored in (bfloat16 widens exactly).
         self.weight = tensors[f"{prefix}.weight"].to(device=device, dtype=torch.float32).contiguous()
+        if params.get("weight_offset"):
+            self.weight = self.weight + float(params["weight_offset"])
         self.groups = int(params.get("groups") or 1)
         if self.size % self.groups:
             raise InvalidArgumentError(f"{prefix}: {self.groups} groups do not divide a row of {self.size}")

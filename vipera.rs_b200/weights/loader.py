@@ -27,6 +27,8 @@ INIT = {
     "embedding": (0.0, 0.02),
     "bias": (0.0, 0.02),
     "norm": (1.0, 0.01),
+    "centred_norm": (0.0, 0.01),   # a norm's weight stored as its distance from one
+    "layer_scale": (1.0, 0.1),     # a number per channel that scales what joins the stream
     "mix": (0.3, 0.4),        # a matrix that mixes heads
     "filter": (0.0, 0.3),     # taps of a short convolution
     "log_rate": (0.0, 0.5),   # logarithms of decay rates
