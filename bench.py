@@ -823,6 +823,68 @@ def fasolorn_decode_bytes(config, batch, history, element=2):
     return {"weights": weights * element, "state": 0, "cache": int(cache)}
 
 
+# ---------------------------------------------------------------------------------------
+# --design nuvezen: the Nuvezen design beside the Qwen2 decoder (or another design) at equal sizes
+# ---------------------------------------------------------------------------------------
+def nuvezen_config(width, heads, kv_heads, ff, layers, vocab, *_unused, experts=16, top=4, window=1024):
+    """`layers` layers of attention over a cached latent of 512 (heads of 128 + 64 turning values, queries
+    through a latent of half the width, at most 1,536, a sink per head, a window); feed-forwards by
+    turns a gated unit of the dense inner size and a mixture of `experts` bounded gated units of which a
+    token uses `top`, beside a gated shared unit, each a fifth of the dense inner size."""
+    mixer = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": min(1536, width // 2),
+             "scale": 192 ** -0.5, "mask": {"size": window}, "rot": {"dims": 64, "base": 10000.0}}
+    piece = ff // (top + 1) // 16 * 16
+    moe = {"kind": "moe", "expert": {"ff": piece, "limit": 7.0}, "shared": {"ff": piece, "limit": 7.0},
+           "router": {"experts": experts, "top": top}}
+    dense = {"kind": "dense", "ff": ff}
+    return {"architecture": "Nuvezen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [{"type": "latent_attention", "mixer": mixer, "mlp": moe if index % 2 else dense} for index in range(layers)]}
+
+
+def nuvezen_work(config, tokens):
+    """Floating-point operations of a prompt of `tokens` tokens by class of kernel (as fasolorn_work)."""
+    width = config["width"]
+    flops = {"proj": 2.0 * config["vocab"] * width, "attention": 0.0, "experts": 0.0}
+    for layer in config["layers"]:
+        m = layer["mixer"]
+        window = m["mask"]["size"] if m.get("mask") else tokens
+        seen = sum(min(position + 1, window) for position in range(tokens))     # (query, key) pairs
+        h, d, r, dv, rank, q_rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+        flops["proj"] += 2.0 * tokens * (width * (q_rank + rank + r + h * dv) + q_rank * h * (d + r))
+        flops["attention"] += 2.0 * h * (seen * (2 * rank + r) + tokens * rank * (d + dv))
+        mlp = layer.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            flops["proj"] += 2.0 * tokens * 3 * width * mlp["ff"]
+        elif mlp:
+            router = mlp["router"]
+            inner = router["top"] * mlp["expert"]["ff"] + (mlp.get("shared") or {"ff": 0})["ff"]
+            flops["experts"] += 2.0 * tokens * (3 * width * inner + (router["experts"] + 1) * width)
+    return flops
+
+
+def nuvezen_decode_bytes(config, batch, history, element=2):
+    """What one decode step must move: every matrix a token of the batch can use (all experts once the
+    batch's choices cover them: min(experts, batch * top)), and the latents within the windows."""
+    width = config["width"]
+    weights = config["vocab"] * width
+    cache = 0
+    for layer in config["layers"]:
+        m = layer["mixer"]
+        keys = min(history, m["mask"]["size"]) if m.get("mask") else history
+        h, d, r, dv, rank, q_rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+        weights += width * (q_rank + rank + r + h * dv) + q_rank * h * (d + r) + h * rank * (d + dv)
+        cache += batch * keys * (rank + r) * element
+        mlp = layer.get("mlp")
+        if mlp and mlp["kind"] == "dense":
+            weights += 3 * width * mlp["ff"]
+        elif mlp:
+            router = mlp["router"]
+            used = min(router["experts"], batch * router["top"])
+            weights += 3 * width * (used * mlp["expert"]["ff"] + (mlp.get("shared") or {"ff": 0})["ff"])
+            weights += (router["experts"] + 1) * width * 2     # the router's matrix is 32-bit
+    return {"weights": weights * element, "state": 0, "cache": int(cache)}
+
+
 DESIGNS = {
     "nobupel": (lambda *sizes: nobupel_config(*sizes), lambda config, tokens: nobupel_work(config, tokens),
                 lambda config, batch, history: nobupel_decode_bytes(config, batch, history)),
@@ -832,6 +894,8 @@ DESIGNS = {
                 lambda config, batch, history: pugovik_decode_bytes(config, batch, history)),
     "fasolorn": (lambda *sizes: fasolorn_config(*sizes), lambda config, tokens: fasolorn_work(config, tokens),
                  lambda config, batch, history: fasolorn_decode_bytes(config, batch, history)),
+    "nuvezen": (lambda *sizes: nuvezen_config(*sizes), lambda config, tokens: nuvezen_work(config, tokens),
+                lambda config, batch, history: nuvezen_decode_bytes(config, batch, history)),
 }
 
 
@@ -870,8 +934,9 @@ def profiled_prefill(model, tokens, page_size):
 
 
 def measure_design(args, peaks, peak_source):
-    """Prefill and decode of the design at sizes that resemble real layers, beside the Qwen2 decoder of
-    the same width, heads, inner size and layer count; random weights, bfloat16."""
+    """Prefill and decode of the design at sizes that resemble real layers, beside the Qwen2 decoder (or,
+    with --beside, another design) of the same width, heads, inner size and layer count; random
+    weights, bfloat16."""
     import torch  # noqa: F401
 
     from vipera_rs_b200.engine import random_model
@@ -885,22 +950,23 @@ def measure_design(args, peaks, peak_source):
         if args.design_size and name != args.design_size:
             continue
         row = {}
-        make_config, work_of, decode_bytes_of = DESIGNS[args.design]
-        for label, config in ((args.design, make_config(width, heads, kv_heads, ff, layers, vocab, cell_heads, cell_dim,
-                                                        cell_vdim)),
-                              ("qwen2", qwen_like(width, heads, kv_heads, ff, layers, vocab))):
+        shape = (width, heads, kv_heads, ff, layers, vocab, cell_heads, cell_dim, cell_vdim)
+        other = qwen_like(*shape[:6]) if args.beside == "qwen2" else DESIGNS[args.beside][0](*shape)
+        for label, config in ((args.design, DESIGNS[args.design][0](*shape)), (args.beside, other)):
+            if label != "qwen2":
+                _, work_of, decode_bytes_of = DESIGNS[label]
             model = random_model(config, seed=0, dtype="bfloat16", device="cuda:0")
             out = {"layers": layers}
             ms = measure_prefill(model, tokens, repeats=5, warmup=3, page_size=args.page_size)
             out["prefill_ms"], out["prefill_tok_s"] = round(ms, 3), round(tokens * 1000.0 / ms, 1)
             out["prefill_ms_by_class"] = profiled_prefill(model, tokens, args.page_size)
-            if label == args.design:
+            if label != "qwen2":
                 work = work_of(config, tokens)
                 out["prefill_flops_by_class"] = {k: round(v / 1e9, 2) for k, v in work.items()}
                 out["prefill_frac_by_class"] = {
                     k: round(v / (out["prefill_ms_by_class"][k] * 1e-3) / (peaks["bf16_tflops"] * 1e12), 4)
                     for k, v in work.items() if out["prefill_ms_by_class"].get(k)}
-                if args.design == "gusolix" and out["prefill_ms_by_class"].get("recurrence"):
+                if label == "gusolix" and out["prefill_ms_by_class"].get("recurrence"):
                     moved = gusolix_prefill_bytes(config, tokens)
                     out["prefill_recurrence_hbm_frac"] = round(
                         moved / (out["prefill_ms_by_class"]["recurrence"] * 1e-3) / 1e9 / peaks["hbm_gbs"], 4)
@@ -914,7 +980,7 @@ def measure_design(args, peaks, peak_source):
                 del harness
                 release_memory()
                 out[f"decode_b{batch}_tok_s"], out[f"decode_b{batch}_ms"] = round(batch * 1000.0 / step_ms, 1), round(step_ms, 4)
-                if label == args.design:
+                if label != "qwen2":
                     moved = decode_bytes_of(config, batch, mean_history)
                     out[f"decode_b{batch}_hbm_frac"] = round(sum(moved.values()) / (step_ms * 1e-3) / 1e9 / peaks["hbm_gbs"], 4)
                 else:
@@ -924,7 +990,7 @@ def measure_design(args, peaks, peak_source):
             del model
             release_memory()
         sizes[name] = row
-    print(json.dumps({"design": args.design, "beside": "qwen2 at equal width, heads, inner size and layers",
+    print(json.dumps({"design": args.design, "beside": f"{args.beside} at equal width, heads, inner size and layers",
                       "dtype": "bf16", "data": "synthetic: seeded random weights, uniform random token ids",
                       "prefill_tokens": tokens, "history": args.history, "steps": args.steps, "warmup": warmup,
                       "peaks": peak_source, "sizes": sizes, "clocks": sampler.stop()}))
@@ -978,6 +1044,8 @@ def main():
     parser.add_argument("--design", choices=sorted(DESIGNS), default=None,
                         help="instead of the headline: prefill and decode of that design at sizes that resemble "
                              "real layers, beside the Qwen2 decoder at equal sizes")
+    parser.add_argument("--beside", choices=["qwen2", *sorted(DESIGNS)], default="qwen2",
+                        help="what --design is measured beside (default: the Qwen2 decoder)")
     parser.add_argument("--design-size", choices=sorted(DESIGN_SIZES), default=None, help="one of the sizes only")
     args = parser.parse_args()
 

@@ -165,10 +165,11 @@ def test_attention_over_latents_with_sinks_and_a_window(name, form, dtype):
     mixed = torch.full((tokens, heads, rank), float("nan"), device=DEV)
     out = torch.full((tokens, heads * dv), float("nan"), dtype=dtype, device=DEV)
     max_keys = max(lengths)
-    floats = ops.latent_part_floats(tokens, heads, rank, max_keys, ops.sm_count(torch.device(DEV)), window)
-    splits = ops.latent_plan(tokens, heads, max_keys, ops.sm_count(torch.device(DEV)), window)[3]
+    single = all(new == 1 for _, new in requests)
+    floats = ops.latent_part_floats(tokens, heads, rank, rot, max_keys, ops.sm_count(torch.device(DEV)), window, single)
+    splits = ops.latent_plan(tokens, heads, rank, rot, max_keys, ops.sm_count(torch.device(DEV)), window, single)[3]
     if window:      # the splits are no more than the window needs, whatever the history
-        assert splits <= ops.latent_plan(tokens, heads, window + 96, ops.sm_count(torch.device(DEV)), 0)[3]
+        assert splits * ops.latent_plan(tokens, heads, rank, rot, max_keys, ops.sm_count(torch.device(DEV)), window, single)[2] <= window + 256
     part = torch.full((floats,), float("nan"), device=DEV) if form != "whole" and floats else None
     buffers = None
     if form == "head_major":
@@ -189,7 +190,7 @@ def test_attention_over_latents_with_sinks_and_a_window(name, form, dtype):
                          token_entry=torch.tensor(entry, dtype=torch.int32, device=DEV), block_table=table.to(DEV),
                          cos=cos.float().to(DEV), sin=sin.float().to(DEV), k_pool=k_pool.to(DEV), v_pool=v_pool.to(DEV), qa=qa,
                          latent_out=mixed, out=out, heads=heads, head_dim=d, rot_dim=rot, value_dim=dv, scale=scale,
-                         max_keys=max_keys, part=part, head_major=buffers, window=window, sink=sink.to(DEV), q=q.to(DEV))
+                         max_keys=max_keys, part=part, head_major=buffers, window=window, sink=sink.to(DEV), q=q.to(DEV), single=single)
     ops.check_kernel_status(torch.device(DEV))
     got = out.cpu().double()
     assert torch.isfinite(got).all()

@@ -541,9 +541,8 @@ def test_the_fold_over_latents_alone(name, cut, head_major):
     mixed = torch.full((tokens, heads, rank), float("nan"), dtype=torch.float32, device=device)
     out = torch.full((tokens, heads * dv), float("nan"), dtype=torch.bfloat16, device=device)
     max_keys = max(lengths)
-    floats = ops.latent_part_floats(tokens, heads, rank, max_keys, ops.sm_count(torch.device(device)))
-    assert floats > 0
-    part = torch.full((floats,), float("nan"), dtype=torch.float32, device=device) if cut else None
+    floats = ops.latent_part_floats(tokens, heads, rank, rot, max_keys, ops.sm_count(torch.device(device)))
+    part = torch.full((floats,), float("nan"), dtype=torch.float32, device=device) if cut and floats else None
     buffers = None
     if head_major:   # the products with the up matrices as grouped tensor-core products, a head a group
         padded = -(-tokens // 128) * 128

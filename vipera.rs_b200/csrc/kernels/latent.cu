@@ -36,8 +36,34 @@ __device__ __forceinline__ void rot_pair(int pairing, int rot, int i, int& a, in
 // block leaves them normed in `cq` [tokens, q_rank], the operand of the product that makes the
 // queries.  kv_off < 0: the layer keeps nothing of its own, only the query latent is normed.
 // ---------------------------------------------------------------------------------------
+// blockIdx.y 0: the cache write, 1: the query latent; each block reads its row once.
+constexpr int kStoreThreads = 128;
+constexpr int kStoreKept = 8;   // values a thread keeps between its two passes: latents up to 1024
+
 template <typename T>
-__global__ void __launch_bounds__(128)
+__device__ __forceinline__ void norm_latent(const float* __restrict__ row, int n, const float* __restrict__ weight, float eps,
+                                            T* __restrict__ dst, float* scratch) {
+  float kept[kStoreKept], gain[kStoreKept], sum = 0.0f;
+#pragma unroll
+  for (int j = 0; j < kStoreKept; ++j) {
+    const int i = threadIdx.x + j * kStoreThreads;
+    kept[j] = i < n ? row[i] : 0.0f;
+    gain[j] = i < n ? weight[i] : 0.0f;
+  }
+#pragma unroll
+  for (int j = 0; j < kStoreKept; ++j) sum += kept[j] * kept[j];
+  for (int i = threadIdx.x + kStoreKept * kStoreThreads; i < n; i += kStoreThreads) sum += row[i] * row[i];
+  const float inverse = 1.0f / sqrtf(block_sum(sum, scratch) / static_cast<float>(n) + eps);
+#pragma unroll
+  for (int j = 0; j < kStoreKept; ++j) {
+    const int i = threadIdx.x + j * kStoreThreads;
+    if (i < n) dst[i] = from_float<T>(kept[j] * inverse * gain[j]);
+  }
+  for (int i = threadIdx.x + kStoreKept * kStoreThreads; i < n; i += kStoreThreads) dst[i] = from_float<T>(row[i] * inverse * weight[i]);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kStoreThreads)
 latent_store_kernel(const float* __restrict__ proj, long long proj_width, int kv_off, const float* __restrict__ norm_weight,
                     float eps, const int* __restrict__ positions, const float* __restrict__ cos_table,
                     const float* __restrict__ sin_table, T* __restrict__ k_pool, T* __restrict__ v_pool,
@@ -48,24 +74,16 @@ latent_store_kernel(const float* __restrict__ proj, long long proj_width, int kv
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
-  if (q_rank > 0) {
-    const float* q_row = proj + static_cast<size_t>(t) * proj_width + cq_off;
-    float squares = 0.0f;
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) squares += q_row[i] * q_row[i];
-    const float inverse = 1.0f / sqrtf(block_sum(squares, scratch) / static_cast<float>(q_rank) + eps);
-    T* dst = cq + static_cast<size_t>(t) * q_rank;
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) dst[i] = from_float<T>(q_row[i] * inverse * cq_norm_weight[i]);
+  const float* row = proj + static_cast<size_t>(t) * proj_width;
+  if (blockIdx.y == 1 || kv_off < 0) {
+    if (q_rank > 0 && (blockIdx.y == 1 || gridDim.y == 1))
+      norm_latent<T>(row + cq_off, q_rank, cq_norm_weight, eps, cq + static_cast<size_t>(t) * q_rank, scratch);
+    return;
   }
-  if (kv_off < 0) return;
-  const float* row = proj + static_cast<size_t>(t) * proj_width + kv_off;
+  row += kv_off;
   const int position = positions[t];
   const int page = block_table[static_cast<size_t>(token_entry[t]) * table_width + position / page_size];
   const size_t slot = static_cast<size_t>(page) * page_size + position % page_size;
-  float sum = 0.0f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) sum += row[i] * row[i];
-  const float inverse = 1.0f / sqrtf(block_sum(sum, scratch) / static_cast<float>(rank) + eps);
-  T* c_row = k_pool + slot * rank;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) c_row[i] = from_float<T>(row[i] * inverse * norm_weight[i]);
   T* r_row = v_pool + slot * rot;
   const float* cs = cos_table + static_cast<size_t>(position) * (rot / 2);
   const float* sn = sin_table + static_cast<size_t>(position) * (rot / 2);
@@ -76,62 +94,141 @@ latent_store_kernel(const float* __restrict__ proj, long long proj_width, int kv
     r_row[ia] = from_float<T>(u * cs[i] - v * sn[i]);
     r_row[ib] = from_float<T>(v * cs[i] + u * sn[i]);
   }
+  norm_latent<T>(row, rank, norm_weight, eps, k_pool + slot * rank, scratch);
 }
 
 // ---------------------------------------------------------------------------------------
 // qa[t, h, :rank] = scale * sum_d q[t, h, d] U[h, d, :],  qa[t, h, rank:] = scale * rotated q.
 // q sits in `proj` at column q_off, head by head as [d unrotated | rot rotated].  U is stored
-// [heads * d, rank].  A block serves kTile tokens of one head, so a row of U is read once per tile.
+// [heads * d, rank].  A block serves kTile tokens of one head and 64 columns, so U is read once per tile.
 // ---------------------------------------------------------------------------------------
 constexpr int kTile = 8;
 
+// acc = A B for up to kTile rows A [kTile][K] (shared memory, transposed: a_t[k * kTile + row]) and COLS
+// columns of B [K, n] (rows of n values, COLS neighbouring ones from `b` on).  A block of eight warps:
+// a lane takes four neighbouring columns, COLS / 4 lanes a row of B, so a warp reads 128 / COLS rows at
+// a time and the eight warps share K between them, all their reads of B in flight together.  The
+// warps' sums are added in their order: on return thread i holds element (i / COLS, i % COLS) of the
+// tile for i < kTile * COLS (and i + 256 where there are more) through `put`.  n and b's column are
+// multiples of 4; columns from `valid` on are not read and come out as 0.
+constexpr int kUpThreads = 256;
+
 template <typename TW>
-__global__ void __launch_bounds__(128)
+__device__ __forceinline__ float4 load_four(const TW* src);
+template <>
+__device__ __forceinline__ float4 load_four<float>(const float* src) { return *reinterpret_cast<const float4*>(src); }
+template <>
+__device__ __forceinline__ float4 load_four<__nv_bfloat16>(const __nv_bfloat16* src) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(src);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
+template <typename TW, int COLS, typename Put>
+__device__ __forceinline__ void tile_product(const float* a_t, const TW* __restrict__ b, int k_count, int n, int valid,
+                                             float* partial /* [8][kTile][COLS] */, Put put) {
+  constexpr int kLanes = COLS / 4, kRowsWarp = 32 / kLanes, kStep = 8 * kRowsWarp;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c4 = (lane % kLanes) * 4, k0 = warp * kRowsWarp + lane / kLanes;
+  float acc[kTile][4];
+#pragma unroll
+  for (int t = 0; t < kTile; ++t)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[t][e] = 0.0f;
+  if (c4 < valid) {
+#pragma unroll 8
+    for (int k = k0; k < k_count; k += kStep) {
+      const float4 w = load_four<TW>(b + static_cast<size_t>(k) * n + c4);
+      const float4 lo = *reinterpret_cast<const float4*>(a_t + k * kTile), hi = *reinterpret_cast<const float4*>(a_t + k * kTile + 4);
+      const float a[kTile] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+#pragma unroll
+      for (int t = 0; t < kTile; ++t) {
+        acc[t][0] = fmaf(a[t], w.x, acc[t][0]);
+        acc[t][1] = fmaf(a[t], w.y, acc[t][1]);
+        acc[t][2] = fmaf(a[t], w.z, acc[t][2]);
+        acc[t][3] = fmaf(a[t], w.w, acc[t][3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int offset = kLanes; offset < 32; offset <<= 1)
+#pragma unroll
+    for (int t = 0; t < kTile; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[t][e] += __shfl_xor_sync(0xffffffffu, acc[t][e], offset);
+  if (lane < kLanes) {
+#pragma unroll
+    for (int t = 0; t < kTile; ++t)
+      *reinterpret_cast<float4*>(partial + (warp * kTile + t) * COLS + c4) = make_float4(acc[t][0], acc[t][1], acc[t][2], acc[t][3]);
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < kTile * COLS; i += kUpThreads) {
+    float sum = partial[i];
+#pragma unroll
+    for (int w = 1; w < 8; ++w) sum += partial[w * kTile * COLS + i];
+    put(i / COLS, i % COLS, sum);
+  }
+}
+
+// A tile's rows into shared memory, transposed: warp w reads row w.
+template <typename Row>
+__device__ __forceinline__ void load_tile_rows(float* a_t, int k_count, int count, Row row) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float* src = row(min(warp, count - 1));
+#pragma unroll 8
+  for (int k = lane; k < k_count; k += 32) a_t[k * kTile + warp] = warp < count ? src[k] : 0.0f;
+}
+
+constexpr int kAbsorbCols = 64;   // columns of the latent a block takes
+
+template <typename TW>
+__global__ void __launch_bounds__(kUpThreads)
 latent_absorb_kernel(const float* __restrict__ proj, long long proj_width, int q_off, const TW* __restrict__ up_k,
                      const int* __restrict__ positions, const float* __restrict__ cos_table,
                      const float* __restrict__ sin_table, float* __restrict__ qa, int num_tokens, int heads, int d,
                      int rank, int rot, float scale, int pairing) {
-  extern __shared__ float q_tile[];   // [kTile][d]
+  extern __shared__ __align__(16) float up_shared[];
+  float* a_t = up_shared;                     // [d][kTile]
+  float* partial = up_shared + d * kTile;     // [8][kTile][kAbsorbCols]
   pdl_launch_dependents();
   pdl_wait();
   const int t0 = blockIdx.x * kTile, h = blockIdx.y;
   const int count = min(kTile, num_tokens - t0);
   const int head_width = d + rot;
-  for (int i = threadIdx.x; i < kTile * d; i += blockDim.x) {
-    const int tt = i / d, e = i % d;
-    q_tile[i] = tt < count ? proj[static_cast<size_t>(t0 + tt) * proj_width + q_off + h * head_width + e] : 0.0f;
+  load_tile_rows(a_t, d, count, [&](int tt) { return proj + static_cast<size_t>(t0 + tt) * proj_width + q_off + h * head_width; });
+  if (blockIdx.z == 0) {
+    for (int i = threadIdx.x; i < count * (rot / 2); i += blockDim.x) {
+      const int tt = i / (rot / 2), pair = i % (rot / 2);
+      const int t = t0 + tt;
+      const float* q_rot = proj + static_cast<size_t>(t) * proj_width + q_off + h * head_width + d;
+      const int position = positions[t];
+      const float c = cos_table[static_cast<size_t>(position) * (rot / 2) + pair];
+      const float s = sin_table[static_cast<size_t>(position) * (rot / 2) + pair];
+      int ia, ib;
+      rot_pair(pairing, rot, pair, ia, ib);
+      const float a = q_rot[ia], b = q_rot[ib];
+      float* dst = qa + (static_cast<size_t>(t) * heads + h) * (rank + rot) + rank;
+      dst[ia] = (a * c - b * s) * scale;
+      dst[ib] = (b * c + a * s) * scale;
+    }
   }
   __syncthreads();
   const TW* u = up_k + static_cast<size_t>(h) * d * rank;
-  // (blocks along z share the rank between them)
-  for (int r = blockIdx.z * blockDim.x + threadIdx.x; r < rank; r += gridDim.z * blockDim.x) {
-    float acc[kTile];
-#pragma unroll
-    for (int tt = 0; tt < kTile; ++tt) acc[tt] = 0.0f;
-#pragma unroll 8
-    for (int e = 0; e < d; ++e) {
-      const float w = to_float<TW>(u[static_cast<size_t>(e) * rank + r]);
-#pragma unroll
-      for (int tt = 0; tt < kTile; ++tt) acc[tt] = fmaf(q_tile[tt * d + e], w, acc[tt]);
-    }
-#pragma unroll
-    for (int tt = 0; tt < kTile; ++tt)
-      if (tt < count) qa[(static_cast<size_t>(t0 + tt) * heads + h) * (rank + rot) + r] = acc[tt] * scale;
+  const int r0 = blockIdx.z * kAbsorbCols;
+  if (rank % 4 == 0) {
+    tile_product<TW, kAbsorbCols>(a_t, u + r0, d, rank, rank - r0, partial, [&](int tt, int c, float sum) {
+      if (tt < count && r0 + c < rank) qa[(static_cast<size_t>(t0 + tt) * heads + h) * (rank + rot) + r0 + c] = sum * scale;
+    });
+    return;
   }
-  if (blockIdx.z != 0) return;
-  for (int i = threadIdx.x; i < count * (rot / 2); i += blockDim.x) {
-    const int tt = i / (rot / 2), pair = i % (rot / 2);
-    const int t = t0 + tt;
-    const float* q_rot = proj + static_cast<size_t>(t) * proj_width + q_off + h * head_width + d;
-    const int position = positions[t];
-    const float c = cos_table[static_cast<size_t>(position) * (rot / 2) + pair];
-    const float s = sin_table[static_cast<size_t>(position) * (rot / 2) + pair];
-    int ia, ib;
-    rot_pair(pairing, rot, pair, ia, ib);
-    const float a = q_rot[ia], b = q_rot[ib];
-    float* dst = qa + (static_cast<size_t>(t) * heads + h) * (rank + rot) + rank;
-    dst[ia] = (a * c - b * s) * scale;
-    dst[ib] = (b * c + a * s) * scale;
+  for (int i = threadIdx.x; i < kTile * kAbsorbCols; i += blockDim.x) {   // ranks that are no whole vectors
+    const int tt = i / kAbsorbCols, r = r0 + i % kAbsorbCols;
+    if (tt >= count || r >= rank) continue;
+    float sum = 0.0f;
+#pragma unroll 8
+    for (int e = 0; e < d; ++e) sum = fmaf(a_t[e * kTile + tt], to_float<TW>(u[static_cast<size_t>(e) * rank + r]), sum);
+    qa[(static_cast<size_t>(t0 + tt) * heads + h) * (rank + rot) + r] = sum * scale;
   }
 }
 
@@ -251,9 +348,10 @@ latent_attention_kernel(const float* __restrict__ qa, float* __restrict__ mixed,
 
 // ---------------------------------------------------------------------------------------
 // The same fold on the tensor cores (bfloat16 caches; mma.sync m16n8k16, 32-bit accumulation).
-// A block owns 16 query rows, a row being a (token, head): `tokens_per_tile` neighbouring tokens
-// by `head_group` heads, all of one request (a tile that spans several requests is folded once per
-// request, the other requests' rows masked).  Keys come 64 at a time as rows [c | kr] of shared
+// A block owns 16 (or 32) query rows, a row being a (token, head) and the rows of a step numbered token
+// by token: `tile_rows` neighbouring rows (whole tokens where the heads allow and rows are few, so that
+// a step of single tokens folds each request's keys once; else as many as the block holds).  A tile
+// that spans several requests is folded once per request, the other requests' rows masked.  Keys come 64 at a time as rows [c | kr] of shared
 // memory, the next tile on its way (cp.async) while this one is used.  Per tile the eight warps
 //   1. each score 8 keys against all 16 rows: S = Q K^T over rank + rot values;
 //   2. each take two rows: running maximum, weights p = exp(s - m) rounded to bfloat16, their sum;
@@ -280,7 +378,7 @@ struct LatentFoldParams {
   float* out;                      // [tokens * heads, rank]
   float* part;                     // splits: [num_splits][tokens * heads][rank + 2]: columns, then m and sum
   int num_tokens, heads, rank, rot, table_width, page_size;
-  int head_group, tokens_per_tile, split_keys, num_splits;
+  int tile_rows, split_keys, num_splits;
   int window;                      // > 0: a row at position p sees keys p - window + 1 .. p
   const float* sink;               // [heads] or null: exp(sink_h) joins the softmax's denominator
   // Head-major form (the products on both sides of the fold run as grouped tensor-core products, a
@@ -315,29 +413,33 @@ latent_fold_kernel(LatentFoldParams p) {
   int* row_s = limit_s + kRows;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   {
-    // everything the copies never write (the columns that pad rank and rot) must read as zero
-    uint4* all = reinterpret_cast<uint4*>(fold_shared);
-    const int vectors = (kRows + 2 * kFoldKeys) * stride * 2 / 16;
-    for (int i = threadIdx.x; i < vectors; i += kFoldThreads) all[i] = make_uint4(0u, 0u, 0u, 0u);
+    // what the copies never write (the columns that pad rank and rot) must read as zero
+    const int pad_a = (rank_pad - p.rank) / 8, pads = pad_a + (width_pad - rank_pad - p.rot) / 8;
+    for (int i = threadIdx.x; i < (kRows + 2 * kFoldKeys) * pads; i += kFoldThreads) {
+      const int row = i / pads, c = i % pads;   // (q_s and k_s follow one another)
+      const int column = c < pad_a ? p.rank + c * 8 : rank_pad + p.rot + (c - pad_a) * 8;
+      *reinterpret_cast<uint4*>(q_s + row * stride + column) = make_uint4(0u, 0u, 0u, 0u);
+    }
   }
   pdl_launch_dependents();
   pdl_wait();
-  const int t0 = (gridDim.x - 1 - blockIdx.x) * p.tokens_per_tile;   // the longest histories of a prompt first
-  const int head0 = blockIdx.y * p.head_group;
-  const int split = blockIdx.z;
+  const int total_rows = p.num_tokens * p.heads;
+  const int row0 = (gridDim.x - 1 - blockIdx.x) * p.tile_rows;   // the longest histories of a prompt first
+  const int rows_here = min(p.tile_rows, total_rows - row0);
+  const int t0 = row0 / p.heads, tokens_here = (row0 + rows_here - 1) / p.heads - t0 + 1;   // at most kRows
+  const int split = blockIdx.y;
   const int width = p.rank + p.rot;
   const int rank_chunks = p.rank / 8, row_chunks = rank_chunks + p.rot / 8;
-  const int total_rows = p.num_tokens * p.heads;
   unsigned done = 0;
   for (;;) {
     int lead = -1;
-    for (int tq = 0; tq < p.tokens_per_tile; ++tq)
-      if (t0 + tq < p.num_tokens && !((done >> tq) & 1u)) { lead = tq; break; }
+    for (int tq = 0; tq < tokens_here; ++tq)
+      if (!((done >> tq) & 1u)) { lead = tq; break; }
     if (lead < 0) break;
     const int entry = p.token_entry[t0 + lead];
     int last_key = -1, first_key = 0x7fffffff;
     unsigned taken = 0;
-    for (int tq = lead; tq < p.tokens_per_tile && t0 + tq < p.num_tokens; ++tq)
+    for (int tq = lead; tq < tokens_here; ++tq)
       if (!((done >> tq) & 1u) && p.token_entry[t0 + tq] == entry) {
         taken |= 1u << tq;
         last_key = max(last_key, p.positions[t0 + tq]);
@@ -347,52 +449,45 @@ latent_fold_kernel(LatentFoldParams p) {
     first_key = p.window > 0 ? max(0, first_key - p.window + 1) : 0;
     __syncthreads();   // the pass before is done with the rows' tables
     if (threadIdx.x < kRows) {
-      const int r = threadIdx.x, tq = r / p.head_group, head = head0 + r % p.head_group;
-      const bool valid = tq < p.tokens_per_tile && ((taken >> tq) & 1u) && head < p.heads;
+      const int r = threadIdx.x, tq = min((row0 + r) / p.heads - t0, 31);
+      const bool valid = r < rows_here && ((taken >> tq) & 1u);
       limit_s[r] = valid ? p.positions[t0 + tq] : -1;
-      row_s[r] = valid ? (t0 + tq) * p.heads + head : -1;
+      row_s[r] = valid ? row0 + r : -1;
       m_s[r] = -INFINITY;
       l_s[r] = 0.0f;
     }
     done |= taken;
     __syncthreads();
-    for (int i = threadIdx.x; i < kRows * width; i += kFoldThreads) {
-      const int r = i / width, c = i % width;
-      float v = 0.0f;
-      if (row_s[r] >= 0) {
-        if (p.qa_heads == nullptr) {
-          v = p.qa[static_cast<size_t>(row_s[r]) * width + c];
-        } else if (c < p.rank) {
-          const int token = row_s[r] / p.heads, head = row_s[r] % p.heads;
-          v = p.scale * p.qa_heads[(static_cast<size_t>(head) * p.padded_tokens + token) * p.rank + c];
-        } else {
-          v = p.q_rot[static_cast<size_t>(row_s[r]) * p.rot + c - p.rank];
-        }
-      }
-      q_s[r * stride + (c < p.rank ? c : rank_pad + c - p.rank)] = __float2bfloat16(v);
-    }
     // first_key is 0 without a window; tiles start at multiples of kFoldKeys either way
     const int begin = first_key / kFoldKeys * kFoldKeys + split * p.split_keys;
     const int end = p.num_splits > 1 ? min(last_key + 1, begin + p.split_keys) : last_key + 1;
     const int num_tiles = end > begin ? (end - begin + kFoldKeys - 1) / kFoldKeys : 0;
+    if (num_tiles == 0) {   // a split that sees no key says so (and leaves no columns); only splits can be such
+      if (threadIdx.x < kRows && row_s[threadIdx.x] >= 0 && p.num_splits > 1) {
+        float* part = p.part + (static_cast<size_t>(split) * total_rows + row_s[threadIdx.x]) * (p.rank + 2);
+        part[p.rank] = -INFINITY;
+        part[p.rank + 1] = 0.0f;
+      }
+      continue;
+    }
     const int* table = p.block_table + static_cast<size_t>(entry) * p.table_width;
 
-    // A warp copies 8 keys of a tile: their page-table entries first (all lanes the same loads, in
-    // flight together), then each row's 16-byte pieces, a lane taking every 32nd.
-    auto copy_tile = [&](int tile) {
+    // A warp copies 8 keys of a tile.  Their places in the pools are looked up a tile ahead, a lane a
+    // key, so that the copies need not wait for the page table; then each row's 16-byte pieces, a lane
+    // taking every 32nd.
+    auto look_up = [&](int tile) {
+      const int key = max(min(begin + tile * kFoldKeys + warp * 8 + (lane & 7), end - 1), first_key);
+      return static_cast<unsigned>(table[key / p.page_size]) * static_cast<unsigned>(p.page_size) + key % p.page_size;
+    };
+    auto copy_tile = [&](int tile, unsigned place) {
       __nv_bfloat16* dst_tile = k_s + (tile & 1) * kFoldKeys * stride;
       const int key0 = begin + tile * kFoldKeys + warp * 8;
-      size_t slots[8];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int key = max(min(key0 + i, end - 1), first_key);
-        slots[i] = static_cast<size_t>(table[key / p.page_size]) * p.page_size + key % p.page_size;
-      }
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const bool valid = key0 + i < end && key0 + i >= first_key;
-        const __nv_bfloat16* c_row = p.k_pool + slots[i] * p.rank;
-        const __nv_bfloat16* r_row = p.v_pool + slots[i] * p.rot;
+        const size_t slot = __shfl_sync(0xffffffffu, place, i);
+        const __nv_bfloat16* c_row = p.k_pool + slot * p.rank;
+        const __nv_bfloat16* r_row = p.v_pool + slot * p.rot;
         __nv_bfloat16* dst = dst_tile + (warp * 8 + i) * stride;
         for (int chunk = lane; chunk < row_chunks; chunk += 32) {
           const bool latent = chunk < rank_chunks;
@@ -413,11 +508,46 @@ latent_fold_kernel(LatentFoldParams p) {
         for (int e = 0; e < 4; ++e) acc[mt][j][e] = 0.0f;
     const int column0 = warp * (NR / 8);
     const int g = lane >> 2, pair = (lane & 3) * 2;
-    if (num_tiles > 0) copy_tile(0);
+    copy_tile(0, look_up(0));
+    unsigned ahead = num_tiles > 1 ? look_up(1) : 0u;
+    // The queries while the first keys are on their way: 8 values at a time, four reads in flight a thread.
+    constexpr int kAtOnce = 4;
+    for (int i0 = threadIdx.x; i0 < kRows * row_chunks; i0 += kAtOnce * kFoldThreads) {
+      float4 lo[kAtOnce], hi[kAtOnce];
+#pragma unroll
+      for (int j = 0; j < kAtOnce; ++j) {
+        const int i = i0 + j * kFoldThreads;
+        const int r = i / row_chunks, c = (i - r * row_chunks) * 8;
+        const int source_row = r < kRows ? row_s[r] : -1;
+        lo[j] = hi[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (source_row >= 0) {
+          const float* src;
+          if (p.qa_heads == nullptr) src = p.qa + static_cast<size_t>(source_row) * width + c;
+          else if (c < p.rank)
+            src = p.qa_heads + (static_cast<size_t>(source_row % p.heads) * p.padded_tokens + source_row / p.heads) * p.rank + c;
+          else src = p.q_rot + static_cast<size_t>(source_row) * p.rot + c - p.rank;
+          lo[j] = *reinterpret_cast<const float4*>(src);
+          hi[j] = *reinterpret_cast<const float4*>(src + 4);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < kAtOnce; ++j) {
+        const int i = i0 + j * kFoldThreads;
+        const int r = i / row_chunks, c = (i - r * row_chunks) * 8;
+        if (r >= kRows) continue;
+        const float f = p.qa_heads != nullptr && c < p.rank ? p.scale : 1.0f;
+        *reinterpret_cast<uint4*>(q_s + r * stride + (c < p.rank ? c : rank_pad + c - p.rank)) =
+            make_uint4(pack_bf16(lo[j].x * f, lo[j].y * f), pack_bf16(lo[j].z * f, lo[j].w * f),
+                       pack_bf16(hi[j].x * f, hi[j].y * f), pack_bf16(hi[j].z * f, hi[j].w * f));
+      }
+    }
     for (int tile = 0; tile < num_tiles; ++tile) {
       cp_async_wait<0>();
       __syncthreads();   // this tile has landed (and the queries, before the first); the tile before is read out
-      if (tile + 1 < num_tiles) copy_tile(tile + 1);
+      if (tile + 1 < num_tiles) {
+        copy_tile(tile + 1, ahead);
+        if (tile + 2 < num_tiles) ahead = look_up(tile + 2);
+      }
       const __nv_bfloat16* keys = k_s + (tile & 1) * kFoldKeys * stride;
       const int key0 = begin + tile * kFoldKeys;
       {
@@ -428,7 +558,7 @@ latent_fold_kernel(LatentFoldParams p) {
           for (int e = 0; e < 4; ++e) c[mt][e] = c_odd[mt][e] = 0.0f;
         const uint32_t k_addr = smem_addr(keys + (warp * 8 + (lane & 7)) * stride + (lane >> 3) * 8);
         const uint32_t q_addr = smem_addr(q_s + ((lane & 7) + ((lane >> 3) & 1) * 8) * stride + (lane >> 4) * 8);
-#pragma unroll 2
+#pragma unroll 3
         for (int k0 = 0; k0 < width_pad; k0 += 32) {
           uint32_t b[4];
           ldmatrix_x4(b, k_addr + k0 * 2);
@@ -452,25 +582,44 @@ latent_fold_kernel(LatentFoldParams p) {
           }
       }
       __syncthreads();
+      {
+        // a warp's rows side by side, so that their reductions fill one another's waits; a lane takes
+        // two neighbouring keys
+        constexpr int kOwn = 2 * MT;
+        const int own0 = warp * kOwn;
+        float2 v[kOwn];
+        float before[kOwn], top[kOwn], sum[kOwn];
 #pragma unroll
-      for (int i = 0; i < 2 * MT; ++i) {
-        const int row = warp * 2 * MT + i;
-        const float v0 = s_s[row * kScoreStride + lane], v1 = s_s[row * kScoreStride + lane + 32];
-        const float before = m_s[row];
-        const float top = fmaxf(before, warp_max(fmaxf(v0, v1)));
-        float alpha = 1.0f, w0 = 0.0f, w1 = 0.0f;
-        if (top > -INFINITY) {
-          alpha = expf(before - top);   // 0 while nothing was seen
-          w0 = __bfloat162float(__float2bfloat16(expf(v0 - top)));
-          w1 = __bfloat162float(__float2bfloat16(expf(v1 - top)));
+        for (int i = 0; i < kOwn; ++i) {
+          v[i] = *reinterpret_cast<const float2*>(s_s + (own0 + i) * kScoreStride + 2 * lane);
+          before[i] = m_s[own0 + i];
+          top[i] = fmaxf(v[i].x, v[i].y);
         }
-        p_s[row * kWeightStride + lane] = __float2bfloat16(w0);
-        p_s[row * kWeightStride + lane + 32] = __float2bfloat16(w1);
-        const float sum = warp_sum(w0 + w1);
-        if (lane == 0) {
-          m_s[row] = top;
-          l_s[row] = l_s[row] * alpha + sum;
-          alpha_s[row] = alpha;
+#pragma unroll
+        for (int offset = 16; offset > 0; offset >>= 1)
+#pragma unroll
+          for (int i = 0; i < kOwn; ++i) top[i] = fmaxf(top[i], __shfl_xor_sync(0xffffffffu, top[i], offset));
+#pragma unroll
+        for (int i = 0; i < kOwn; ++i) {
+          top[i] = fmaxf(top[i], before[i]);
+          const float shift = top[i] > -INFINITY ? top[i] : 0.0f;   // (a row that has seen nothing: e^(-inf) = 0)
+          const __nv_bfloat162 w = __floats2bfloat162_rn(expf(v[i].x - shift), expf(v[i].y - shift));
+          *reinterpret_cast<__nv_bfloat162*>(p_s + (own0 + i) * kWeightStride + 2 * lane) = w;
+          const float2 rounded = __bfloat1622float2(w);
+          sum[i] = rounded.x + rounded.y;
+        }
+#pragma unroll
+        for (int offset = 16; offset > 0; offset >>= 1)
+#pragma unroll
+          for (int i = 0; i < kOwn; ++i) sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], offset);
+#pragma unroll
+        for (int i = 0; i < kOwn; ++i) {
+          if (lane == i) {
+            const float alpha = top[i] > -INFINITY ? expf(before[i] - top[i]) : 1.0f;   // 0 while nothing was seen
+            m_s[own0 + i] = top[i];
+            l_s[own0 + i] = l_s[own0 + i] * alpha + sum[i];
+            alpha_s[own0 + i] = alpha;
+          }
         }
       }
       __syncthreads();
@@ -549,54 +698,82 @@ latent_fold_kernel(LatentFoldParams p) {
   }
 }
 
-// out[row, :] = sum_s e^(m_s - m) columns_s / sum_s e^(m_s - m) sum_s over the splits that saw a key.
-// The splits' maxima and sums are read side by side (a thread a split), the weights e^(m_s - m) / total
-// kept in shared memory, and a column's terms asked for four splits at a time, added in the splits' order.
+// out[row, :] = sum_s e^(m_s - m) columns_s / sum_s e^(m_s - m) sum_s over the splits that saw a key
+// (the others left no columns).  The first warp reads the splits' maxima and sums side by side and lists
+// the splits that count with their weights e^(m_s - m) / total; a column's terms are asked for eight
+// splits at a time and added in the splits' order.
 constexpr int kMostSplits = 64;
 
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(LatentFoldParams p) {
-  __shared__ float top_s[kMostSplits], sum_s[kMostSplits], weight_s[kMostSplits];
+  __shared__ float weight_s[kMostSplits];
+  __shared__ int split_s[kMostSplits];
+  __shared__ int counted;
   pdl_launch_dependents();
   pdl_wait();
   const int row = blockIdx.x;
   const size_t rows = static_cast<size_t>(p.num_tokens) * p.heads, each = p.rank + 2;
   const float* first = p.part + static_cast<size_t>(row) * each;
-  if (threadIdx.x < p.num_splits) {
-    const float* part = first + threadIdx.x * rows * each;
-    top_s[threadIdx.x] = part[p.rank];
-    sum_s[threadIdx.x] = part[p.rank + 1];
-  }
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    float top = -INFINITY, total = 0.0f;
-    for (int s = 0; s < p.num_splits; ++s)
-      if (sum_s[s] > 0.0f) top = fmaxf(top, top_s[s]);
-    for (int s = 0; s < p.num_splits; ++s) {
-      weight_s[s] = sum_s[s] > 0.0f ? expf(top_s[s] - top) : 0.0f;
-      total += sum_s[s] * weight_s[s];
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    float top[2], sum[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int split = lane + 32 * j;
+      const float* part = first + static_cast<size_t>(min(split, p.num_splits - 1)) * rows * each;
+      sum[j] = split < p.num_splits ? part[p.rank + 1] : 0.0f;
+      top[j] = sum[j] > 0.0f ? part[p.rank] : -INFINITY;
     }
-    if (p.sink) total += expf(p.sink[row % p.heads] - top);
+    const float most = warp_max(fmaxf(top[0], top[1]));
+    float weight[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) weight[j] = sum[j] > 0.0f ? expf(top[j] - most) : 0.0f;
+    float total = warp_sum(sum[0] * weight[0] + sum[1] * weight[1]);
+    if (p.sink) total += expf(p.sink[row % p.heads] - most);
     const float inverse = 1.0f / total;
-    for (int s = 0; s < p.num_splits; ++s) weight_s[s] *= inverse;
+    int base = 0;
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const unsigned live = __ballot_sync(0xffffffffu, sum[j] > 0.0f);
+      if (sum[j] > 0.0f) {
+        const int at = base + __popc(live & ((1u << lane) - 1u));
+        split_s[at] = lane + 32 * j;
+        weight_s[at] = weight[j] * inverse;
+      }
+      base += __popc(live);
+    }
+    if (lane == 0) counted = base;
   }
   __syncthreads();
-  for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
-    float sum = 0.0f;
-    int s = 0;
-    for (; s + 4 <= p.num_splits; s += 4) {
-      const float v0 = first[(s * rows) * each + c], v1 = first[((s + 1) * rows) * each + c];
-      const float v2 = first[((s + 2) * rows) * each + c], v3 = first[((s + 3) * rows) * each + c];
-      sum = fmaf(v0, weight_s[s], sum);
-      sum = fmaf(v1, weight_s[s + 1], sum);
-      sum = fmaf(v2, weight_s[s + 2], sum);
-      sum = fmaf(v3, weight_s[s + 3], sum);
+  const int splits = counted;
+  // two neighbouring columns to a thread where rows are whole pairs (`each` is even with the rank)
+  const bool pairs = (p.rank & 1) == 0;
+  for (int c = threadIdx.x * 2; c < p.rank; c += 2 * blockDim.x) {
+    float sum0 = 0.0f, sum1 = 0.0f;
+    for (int s0 = 0; s0 < splits; s0 += 8) {
+      float2 v[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float* part = first + static_cast<size_t>(split_s[min(s0 + i, splits - 1)]) * rows * each + c;
+        if (pairs) v[i] = *reinterpret_cast<const float2*>(part);
+        else v[i] = make_float2(part[0], c + 1 < p.rank ? part[1] : 0.0f);
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (s0 + i < splits) {
+          sum0 = fmaf(v[i].x, weight_s[s0 + i], sum0);
+          sum1 = fmaf(v[i].y, weight_s[s0 + i], sum1);
+        }
     }
-    for (; s < p.num_splits; ++s) sum = fmaf(first[(s * rows) * each + c], weight_s[s], sum);
-    if (p.l_heads != nullptr)
-      p.l_heads[(static_cast<size_t>(row % p.heads) * p.padded_tokens + row / p.heads) * p.rank + c] = __float2bfloat16(sum);
-    else
-      p.out[static_cast<size_t>(row) * p.rank + c] = sum;
+    if (p.l_heads != nullptr) {
+      __nv_bfloat16* dst = p.l_heads + (static_cast<size_t>(row % p.heads) * p.padded_tokens + row / p.heads) * p.rank + c;
+      dst[0] = __float2bfloat16(sum0);
+      if (c + 1 < p.rank) dst[1] = __float2bfloat16(sum1);
+    } else {
+      float* dst = p.out + static_cast<size_t>(row) * p.rank + c;
+      dst[0] = sum0;
+      if (c + 1 < p.rank) dst[1] = sum1;
+    }
   }
 }
 
@@ -652,57 +829,46 @@ latent_gate_kernel(const float* __restrict__ o_heads, const float* __restrict__ 
 }
 
 // ---------------------------------------------------------------------------------------
-// out[t, h * dv + v] = (sum_r l[t, h, r] V[h, r, v]) * sigmoid(gate[t, h * dv + v]).  V is stored
+// out[t, h * dv + v] = (sum_r l[t, h, r] V[h, r, v]) * sigmoid(gate[t, h * dv + v]); a block: kTile tokens of
+// one head, 32 values.  V is stored
 // transposed per head, [heads, rank, dv], so that neighbouring threads read neighbouring values.
 // `gate` is the pre-activation in `proj` at column g_off (g_off < 0: no gate).
 // ---------------------------------------------------------------------------------------
+constexpr int kExpandCols = 32;   // values of a head a block takes
+
 template <typename TW, typename TO>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kUpThreads)
 latent_expand_kernel(const float* __restrict__ latent_out, const TW* __restrict__ up_v, const float* __restrict__ proj,
                      long long proj_width, int g_off, TO* __restrict__ out, int num_tokens, int heads, int dv,
                      int rank) {
-  // A block: kTile tokens of one head, 32 values; its four warps share the rank between them and
-  // add their parts in the warps' order.
-  extern __shared__ float expand_shared[];
-  float* l_tile = expand_shared;                 // [kTile][rank]
-  float* partial = expand_shared + kTile * rank; // [4][kTile][32]
+  extern __shared__ __align__(16) float up_shared[];
+  float* a_t = up_shared;                       // [rank][kTile]
+  float* partial = up_shared + rank * kTile;    // [8][kTile][kExpandCols]
   pdl_launch_dependents();
   pdl_wait();
   const int t0 = blockIdx.x * kTile, h = blockIdx.y;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int v = blockIdx.z * 32 + lane;
   const int count = min(kTile, num_tokens - t0);
-  for (int i = threadIdx.x; i < kTile * rank; i += blockDim.x) {
-    const int tt = i / rank, r = i % rank;
-    l_tile[i] = tt < count ? latent_out[(static_cast<size_t>(t0 + tt) * heads + h) * rank + r] : 0.0f;
-  }
+  load_tile_rows(a_t, rank, count, [&](int tt) { return latent_out + (static_cast<size_t>(t0 + tt) * heads + h) * rank; });
   __syncthreads();
   const TW* w = up_v + static_cast<size_t>(h) * rank * dv;
-  const int share = (rank + 3) / 4;
-  const int r_end = min(rank, (warp + 1) * share);
-  float acc[kTile];
-#pragma unroll
-  for (int tt = 0; tt < kTile; ++tt) acc[tt] = 0.0f;
-  if (v < dv) {
-#pragma unroll 8
-    for (int r = warp * share; r < r_end; ++r) {
-      const float x = to_float<TW>(w[static_cast<size_t>(r) * dv + v]);
-#pragma unroll
-      for (int tt = 0; tt < kTile; ++tt) acc[tt] = fmaf(l_tile[tt * rank + r], x, acc[tt]);
-    }
-  }
-#pragma unroll
-  for (int tt = 0; tt < kTile; ++tt) partial[(warp * kTile + tt) * 32 + lane] = acc[tt];
-  __syncthreads();
-  for (int i = threadIdx.x; i < kTile * 32; i += blockDim.x) {
-    const int tt = i / 32, column = blockIdx.z * 32 + i % 32;
-    if (tt >= count || column >= dv) continue;
-    float y = partial[i];
-#pragma unroll
-    for (int part = 1; part < 4; ++part) y += partial[part * kTile * 32 + i];
+  const int v0 = blockIdx.z * kExpandCols;
+  auto put = [&](int tt, int c, float y) {
+    if (tt >= count || v0 + c >= dv) return;
     const size_t t = t0 + tt;
-    if (g_off >= 0) y *= 1.0f / (1.0f + expf(-proj[t * proj_width + g_off + h * dv + column]));
-    out[(t * heads + h) * dv + column] = from_float<TO>(y);
+    if (g_off >= 0) y *= 1.0f / (1.0f + expf(-proj[t * proj_width + g_off + h * dv + v0 + c]));
+    out[(t * heads + h) * dv + v0 + c] = from_float<TO>(y);
+  };
+  if (dv % 4 == 0) {
+    tile_product<TW, kExpandCols>(a_t, w + v0, rank, dv, dv - v0, partial, put);
+    return;
+  }
+  for (int i = threadIdx.x; i < kTile * kExpandCols; i += blockDim.x) {
+    const int tt = i / kExpandCols, c = i % kExpandCols;
+    if (tt >= count || v0 + c >= dv) continue;
+    float sum = 0.0f;
+#pragma unroll 8
+    for (int r = 0; r < rank; ++r) sum = fmaf(a_t[r * kTile + tt], to_float<TW>(w[static_cast<size_t>(r) * dv + v0 + c]), sum);
+    put(tt, c, sum);
   }
 }
 
@@ -749,43 +915,58 @@ struct LatentParams {
   int cq_off, q_rank;
   const float* cq_norm_weight;   // [q_rank]
   void* cq;                      // [tokens, q_rank], the run's type
+  int single;              // 1: every request of the step brings one token
 };
 
-// How the tensor-core fold cuts a step: {tokens per tile, heads per tile, keys per split, splits}.
-// Few blocks (decode) are cut along the keys, in whole tiles of 64, until the device has some
-// four blocks per SM.
-// Groups of sixteen rows a block takes: two where single groups would still fill the device twice.
-static int fold_groups(int tokens, int heads, int sms) {
-  const int head_group = heads < kFoldRows ? heads : kFoldRows;
-  const int per_tile = kFoldRows / head_group;
-  const long base = static_cast<long>((tokens + per_tile - 1) / per_tile) * ((heads + head_group - 1) / head_group);
-  return base >= 2L * sms && heads <= kFoldRows ? 2 : 1;
+// How the tensor-core fold cuts a step.  Rows are tokens x heads.  Many rows: two groups of sixteen to a
+// block.  Few rows (decode) are cut along the keys besides, in whole tiles of 64; whole tokens to a
+// block then, one at a time where every request brings one token (`single`), so that no block folds
+// the keys of two requests one behind the other.
+struct FoldPlan { int groups, tile_rows, tiles, split_keys, num_splits; };
+
+static size_t fold_shared_bytes(int rank, int rot, int groups) {
+  const int rank_pad = round_up(rank, 16), rows = kFoldRows * groups;
+  const int stride = round_up(rank_pad + round_up(rot, 16), 32) + 8;
+  return static_cast<size_t>(rows + 2 * kFoldKeys) * stride * 2 + rows * kScoreStride * 4 + rows * kWeightStride * 2 + rows * 5 * 4;
 }
 
-static void latent_plan(int tokens, int heads, int max_keys, int window, int sms, int* plan) {
-  const int head_group = heads < kFoldRows ? heads : kFoldRows;
-  const int per_tile = kFoldRows * fold_groups(tokens, heads, sms) / head_group;
-  const long base = static_cast<long>((tokens + per_tile - 1) / per_tile) * ((heads + head_group - 1) / head_group);
-  // with a window a tile's rows together see window + per_tile - 1 keys at most, counted from the
-  // start of a tile of keys
-  if (window > 0 && max_keys > window + per_tile + kFoldKeys) max_keys = window + per_tile + kFoldKeys;
+static FoldPlan latent_plan(int tokens, int heads, int rank, int rot, int max_keys, int window, int single, int sms) {
+  FoldPlan plan{};
+  const long rows = static_cast<long>(tokens) * heads;
+  const bool many = rows >= 2L * sms * kFoldRows && !single;
+  plan.groups = many || (heads > kFoldRows && single) ? 2 : 1;
+  const int most = kFoldRows * plan.groups;
+  plan.tile_rows = most;
+  if (!many && heads <= most) plan.tile_rows = single ? heads : most / heads * heads;
+  plan.tiles = static_cast<int>((rows + plan.tile_rows - 1) / plan.tile_rows);
+  // histories grow from step to step: the cut changes with powers of two only.  With a window a tile's
+  // rows together see fewer than window + 32 keys, counted from the start of a tile of keys.
   int bound = kFoldKeys;
   while (bound < max_keys) bound *= 2;
-  long want = (4L * sms) / base;
-  if (want > bound / kFoldKeys) want = bound / kFoldKeys;
-  if (want > 64) want = 64;
-  if (want < 1) want = 1;
-  int chunk = static_cast<int>((bound + want - 1) / want);
-  chunk = (chunk + kFoldKeys - 1) / kFoldKeys * kFoldKeys;
-  plan[0] = per_tile;
-  plan[1] = head_group;
-  plan[2] = chunk;
-  plan[3] = (bound + chunk - 1) / chunk;
+  if (window > 0) bound = std::min(bound, round_up(window + 32 + kFoldKeys, kFoldKeys));
+  const int key_tiles = bound / kFoldKeys;
+  const int per_sm = static_cast<int>(std::min<size_t>(2, 227 * 1024 / (fold_shared_bytes(rank, rot, plan.groups) + 1024)));
+  const long at_once = static_cast<long>(sms) * std::max(per_sm, 1);
+  plan.num_splits = 1, plan.split_keys = bound;
+  // (waves of blocks) x (tiles of keys in a row + what a block costs besides), the smallest
+  double best = 0.0;
+  for (int splits = 1; splits <= std::min(key_tiles, 64); ++splits) {
+    const int each = (key_tiles + splits - 1) / splits;
+    if (splits > 1 && (key_tiles + each - 1) / each != splits) continue;
+    const double cost = static_cast<double>((plan.tiles * static_cast<long>(splits) + at_once - 1) / at_once) * (each + 2.0) + (splits > 1 ? 1.0 + 0.1 * splits : 0.0);
+    if (splits == 1 || cost < best) best = cost, plan.num_splits = splits, plan.split_keys = each * kFoldKeys;
+  }
+  return plan;
 }
 
-VIPERA_API int vipera_latent_plan(int tokens, int heads, int max_keys, int window, int sms, int* plan) {
-  if (tokens <= 0 || heads <= 0 || sms <= 0 || window < 0) return VIPERA_BAD_ARGUMENT;
-  latent_plan(tokens, heads, max_keys < 1 ? 1 : max_keys, window, sms, plan);
+// {rows of a tile, groups of sixteen rows, keys per split, splits}
+VIPERA_API int vipera_latent_plan(int tokens, int heads, int rank, int rot, int max_keys, int window, int single, int sms, int* plan) {
+  if (tokens <= 0 || heads <= 0 || sms <= 0 || window < 0 || rank <= 0 || rot <= 0) return VIPERA_BAD_ARGUMENT;
+  const FoldPlan f = latent_plan(tokens, heads, rank, rot, max_keys < 1 ? 1 : max_keys, window, single, sms);
+  plan[0] = f.tile_rows;
+  plan[1] = f.groups;
+  plan[2] = f.split_keys;
+  plan[3] = f.num_splits;
   return VIPERA_OK;
 }
 
@@ -821,19 +1002,15 @@ static int launch_fold_any(const LatentParams& p, cudaStream_t s) {
   int device = 0, sms = 0;
   cudaGetDevice(&device);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
-  const int groups = fold_groups(p.num_tokens, p.heads, sms > 0 ? sms : 148);
-  f.head_group = p.heads < kFoldRows ? p.heads : kFoldRows;
-  f.tokens_per_tile = kFoldRows * groups / f.head_group;
+  const FoldPlan plan = latent_plan(p.num_tokens, p.heads, p.rank, p.rot, 1, p.window, p.single, sms > 0 ? sms : 148);
+  const int groups = plan.groups;   // (rows and tiles do not depend on the keys)
+  f.tile_rows = plan.tile_rows;
   f.num_splits = p.num_splits > 1 && p.part ? p.num_splits : 1;
   f.split_keys = f.num_splits > 1 ? p.split_keys : 0x3fffffff;
   if (f.num_splits > kMostSplits) return VIPERA_BAD_ARGUMENT;
   const int rank_pad = round_up(p.rank, 16);
-  const int stride = round_up(rank_pad + round_up(p.rot, 16), 32) + 8;
-  const int rows = kFoldRows * groups;
-  const size_t shared = static_cast<size_t>(rows + 2 * kFoldKeys) * stride * 2 + rows * kScoreStride * 4 +
-                        rows * kWeightStride * 2 + rows * 5 * 4;
-  const dim3 grid((p.num_tokens + f.tokens_per_tile - 1) / f.tokens_per_tile, (p.heads + f.head_group - 1) / f.head_group,
-                  f.num_splits);
+  const size_t shared = fold_shared_bytes(p.rank, p.rot, groups);
+  const dim3 grid(plan.tiles, f.num_splits);
   int status;
   if (groups == 2)
     status = rank_pad <= 128 ? launch_fold<128, 2>(f, grid, shared, s)
@@ -855,10 +1032,11 @@ static int launch_latent(const LatentParams& p, cudaStream_t s) {
                          p.proj_width, p.g_off, static_cast<T*>(p.out), p.num_tokens, p.heads, p.dv, p.padded_tokens);
   }
   if (p.kv_off >= 0 || p.stage == 4) {
-    status = vipera_launch(latent_store_kernel<T>, p.num_tokens, 128, 0, s, p.proj, p.proj_width, p.kv_off, p.norm_weight,
+    const int cq_rank = p.stage == 4 ? p.q_rank : 0;
+    status = vipera_launch(latent_store_kernel<T>, dim3(p.num_tokens, p.kv_off >= 0 && cq_rank > 0 ? 2 : 1), kStoreThreads, 0, s, p.proj, p.proj_width, p.kv_off, p.norm_weight,
                            p.eps, p.positions, p.cos_table, p.sin_table, static_cast<T*>(p.k_pool),
                            static_cast<T*>(p.v_pool), p.token_entry, p.block_table, p.table_width, p.page_size, p.rank,
-                           p.rot, p.pairing, p.cq_off, p.stage == 4 ? p.q_rank : 0, p.cq_norm_weight, static_cast<T*>(p.cq));
+                           p.rot, p.pairing, p.cq_off, cq_rank, p.cq_norm_weight, static_cast<T*>(p.cq));
     if (status || p.stage == 4) return status;
   }
   const float* q = p.q ? p.q : p.proj;
@@ -868,8 +1046,8 @@ static int launch_latent(const LatentParams& p, cudaStream_t s) {
                          p.sin_table, static_cast<__nv_bfloat16*>(p.a_heads), p.q_rot, p.tile_group, p.heads, p.d, p.rot,
                          p.padded_tokens, p.scale, p.pairing);
   const dim3 tiles((p.num_tokens + kTile - 1) / kTile, p.heads);
-  const dim3 absorb_grid(tiles.x, tiles.y, (p.rank + 127) / 128);
-  status = vipera_launch(latent_absorb_kernel<T>, absorb_grid, 128, kTile * p.d * sizeof(float), s, q, q_width, p.q_off,
+  const dim3 absorb_grid(tiles.x, tiles.y, (p.rank + kAbsorbCols - 1) / kAbsorbCols);
+  status = vipera_launch(latent_absorb_kernel<T>, absorb_grid, kUpThreads, (kTile * p.d + 8 * kTile * kAbsorbCols) * sizeof(float), s, q, q_width, p.q_off,
                          static_cast<const T*>(p.up_k), p.positions, p.cos_table, p.sin_table, p.qa, p.num_tokens,
                          p.heads, p.d, p.rank, p.rot, p.scale, p.pairing);
   if (status) return status;
@@ -883,8 +1061,8 @@ static int launch_latent(const LatentParams& p, cudaStream_t s) {
                            static_cast<const T*>(p.k_pool), static_cast<const T*>(p.v_pool), p.token_entry, p.positions,
                            p.block_table, p.table_width, p.page_size, p.heads, p.rank, p.rot, p.window, p.sink);
   if (status) return status;
-  const dim3 expand_grid(tiles.x, tiles.y, (p.dv + 31) / 32);
-  return vipera_launch(latent_expand_kernel<T, T>, expand_grid, 128, (kTile * p.rank + 4 * kTile * 32) * sizeof(float), s, p.latent_out,
+  const dim3 expand_grid(tiles.x, tiles.y, (p.dv + kExpandCols - 1) / kExpandCols);
+  return vipera_launch(latent_expand_kernel<T, T>, expand_grid, kUpThreads, (kTile * p.rank + 8 * kTile * kExpandCols) * sizeof(float), s, p.latent_out,
                        static_cast<const T*>(p.up_v), p.proj, p.proj_width, p.g_off, static_cast<T*>(p.out),
                        p.num_tokens, p.heads, p.dv, p.rank);
 }

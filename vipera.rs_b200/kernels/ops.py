@@ -1574,23 +1574,26 @@ class _LatentParams(ctypes.Structure):
         ("stage", _c_int), ("padded_tokens", _c_int), ("a_heads", _c_void), ("qa_heads", _c_void), ("q_rot", _c_void),
         ("l_heads", _c_void), ("o_heads", _c_void), ("tile_group", _c_void),
         ("window", _c_int), ("pairing", _c_int), ("sink", _c_void), ("q", _c_void), ("q_width", ctypes.c_longlong),
-        ("cq_off", _c_int), ("q_rank", _c_int), ("cq_norm_weight", _c_void), ("cq", _c_void),
+        ("cq_off", _c_int), ("q_rank", _c_int), ("cq_norm_weight", _c_void), ("cq", _c_void), ("single", _c_int),
     ]
 
 
 @functools.lru_cache(maxsize=4096)
-def latent_plan(tokens: int, heads: int, max_keys: int, sm_count: int, window: int = 0):
-    """How the tensor-core fold over the latents cuts a step: (tokens per tile, heads per tile,
-    keys per split, splits).  With a window the splits cover the window only."""
-    fn = _function("latent", "vipera_latent_plan", [_c_int] * 5 + [ctypes.POINTER(_c_int)])
+def latent_plan(tokens: int, heads: int, rank: int, rot: int, max_keys: int, sm_count: int, window: int = 0, single: bool = False):
+    """How the tensor-core fold over the latents cuts a step: ((token, head) rows of a tile, groups of
+    sixteen rows of a block, keys per split, splits).  With a window the splits cover the window only;
+    ``single``: every request of the step brings one token."""
+    fn = _function("latent", "vipera_latent_plan", [_c_int] * 8 + [ctypes.POINTER(_c_int)])
     plan = (_c_int * 4)()
-    _check(fn(int(tokens), int(heads), int(max_keys), int(window or 0), int(sm_count), plan), "latent_plan", kernels=0)
+    _check(fn(int(tokens), int(heads), int(rank), int(rot), int(max_keys), int(window or 0), int(bool(single)), int(sm_count), plan),
+           "latent_plan", kernels=0)
     return tuple(plan)
 
 
-def latent_part_floats(tokens: int, heads: int, rank: int, max_keys: int, sm_count: int, window: int = 0) -> int:
+def latent_part_floats(tokens: int, heads: int, rank: int, rot: int, max_keys: int, sm_count: int, window: int = 0,
+                       single: bool = False) -> int:
     """Floats of scratch the fold's splits need for a step (0 when it runs without splits)."""
-    splits = latent_plan(tokens, heads, max_keys, sm_count, window)[3]
+    splits = latent_plan(tokens, heads, rank, rot, max_keys, sm_count, window, single)[3]
     return splits * tokens * heads * (rank + 2) if splits > 1 else 0
 
 
@@ -1601,7 +1604,7 @@ def latent_attention(proj: torch.Tensor, *, q_off: int, g_off: int, kv_off: int,
                      head_dim: int, rot_dim: int, value_dim: int, scale: float, max_keys: int = 0,
                      part: Optional[torch.Tensor] = None, head_major: Optional[dict] = None, window: int = 0,
                      pairing: int = ROPE_INTERLEAVED, sink: Optional[torch.Tensor] = None,
-                     q: Optional[torch.Tensor] = None) -> None:
+                     q: Optional[torch.Tensor] = None, single: bool = False) -> None:
     """Causal softmax attention whose keys and values are products of a cached latent.  ``proj``
     float32 [tokens, width] holds q (head by head [head_dim | rot_dim]) at column ``q_off``, the
     output gate's pre-activation at ``g_off`` (negative: no gate) and the down projection
@@ -1623,7 +1626,8 @@ def latent_attention(proj: torch.Tensor, *, q_off: int, g_off: int, kv_off: int,
     ROPE_INTERLEAVED (2i, 2i + 1) or ROPE_NEOX (i, i + rot_dim / 2).  ``sink`` (float32 [heads]):
     exp(sink_h) joins the softmax's denominator.  ``q`` (float32 [tokens, heads * (head_dim +
     rot_dim)]): the queries, where they are no columns of ``proj`` (``q_off`` is then a column of q);
-    the cache is then written ahead of this call, by latent_store, and ``kv_off`` is negative."""
+    the cache is then written ahead of this call, by latent_store, and ``kv_off`` is negative.
+    ``single``: every request of the step brings one token (as latent_part_floats was told)."""
     fn = _function("latent", "vipera_latent_attention", [ctypes.POINTER(_LatentParams), _c_int, _c_void])
     _check_struct("latent", "vipera_latent_params_size", _LatentParams)
     tokens = proj.shape[0]
@@ -1667,9 +1671,9 @@ def latent_attention(proj: torch.Tensor, *, q_off: int, g_off: int, kv_off: int,
     if pairing not in (ROPE_INTERLEAVED, ROPE_NEOX):
         raise InvalidArgumentError("latent_attention: the rotated part turns as interleaved pairs or as halves")
     p.window, p.pairing = int(window or 0), 1 if pairing == ROPE_NEOX else 0
-    p.part, p.split_keys, p.num_splits = None, 0, 1
+    p.part, p.split_keys, p.num_splits, p.single = None, 0, 1, int(bool(single))
     if part is not None and max_keys > 0:
-        _, _, split_keys, splits = latent_plan(tokens, heads, int(max_keys), sm_count(proj.device), p.window)
+        _, _, split_keys, splits = latent_plan(tokens, heads, rank, rot_dim, int(max_keys), sm_count(proj.device), p.window, single)
         if splits > 1:
             if part.numel() < splits * tokens * heads * (rank + 2):
                 raise InvalidArgumentError("latent_attention: the scratch of the splits is too small")

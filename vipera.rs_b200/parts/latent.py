@@ -157,7 +157,9 @@ class LatentAttention(Mixer):
         mixed = ws.get("latent.out", (count, self.heads * self.vdim), ctx.dtype)
         cos, sin = self.position.tables()
         max_keys = max(int(ctx.max_kv_len), 1)
-        floats = ops.latent_part_floats(count, self.heads, self.rank, max_keys, ops.sm_count(h.device), self.window) if ctx.dtype == torch.bfloat16 else 0
+        single = bool(ctx.all_single)
+        floats = ops.latent_part_floats(count, self.heads, self.rank, self.rot, max_keys, ops.sm_count(h.device), self.window,
+                                        single) if ctx.dtype == torch.bfloat16 else 0
         part = ws.get("latent.part", (floats,), torch.float32) if floats else None
         head_major = None
         if self.head_major and count >= HEAD_MAJOR_FROM:
@@ -188,7 +190,7 @@ class LatentAttention(Mixer):
                              k_pool=cache.k, v_pool=cache.v, qa=qa, latent_out=mixed_latent, out=mixed, heads=self.heads,
                              head_dim=self.dim, rot_dim=self.rot, value_dim=self.vdim, scale=self.scale, max_keys=max_keys,
                              part=part, head_major=head_major, window=self.window, pairing=self.position.style,
-                             sink=self.sink, q=q)
+                             sink=self.sink, q=q, single=single)
         if residual is None:
             rows = ws.get("latent.rows", (count, self.hidden), torch.float32)
             self.out(ctx, mixed, epilogue=ops.EPI_STORE, out=rows)
