@@ -953,7 +953,10 @@ static FoldPlan latent_plan(int tokens, int heads, int rank, int rot, int max_ke
   for (int splits = 1; splits <= std::min(key_tiles, 64); ++splits) {
     const int each = (key_tiles + splits - 1) / splits;
     if (splits > 1 && (key_tiles + each - 1) / each != splits) continue;
-    const double cost = static_cast<double>((plan.tiles * static_cast<long>(splits) + at_once - 1) / at_once) * (each + 2.0) + (splits > 1 ? 1.0 + 0.1 * splits : 0.0);
+    // (the splits' partial sums stay within 1,300 groups of sixteen rows, which memory is planned for)
+    if (splits > 1 && static_cast<long>(plan.tiles) * splits * plan.groups > 1300) break;
+    const double waves = static_cast<double>((plan.tiles * static_cast<long>(splits) + at_once - 1) / at_once);
+    const double cost = waves * (each + 2.0) + (splits > 1 ? 1.0 + 0.1 * splits : 0.0);
     if (splits == 1 || cost < best) best = cost, plan.num_splits = splits, plan.split_keys = each * kFoldKeys;
   }
   return plan;
