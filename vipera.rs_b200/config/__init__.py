@@ -24,6 +24,7 @@ from .gusolix import GusolixConfig, gusolix_model_spec
 from .pugovik import PugovikConfig, pugovik_model_spec
 from .fasolorn import FasolornConfig, fasolorn_model_spec
 from .nuvezen import NuvezenConfig, nuvezen_model_spec
+from .zugutar import ZugutarConfig, zugutar_model_spec
 
 
 def read_config_json(model_dir: str) -> Dict[str, Any]:
@@ -69,6 +70,6 @@ __all__ = [
     "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry",
     "Qwen2Config", "qwen2_model_spec", "NobupelConfig", "nobupel_model_spec", "GusolixConfig", "gusolix_model_spec",
     "PugovikConfig", "pugovik_model_spec", "FasolornConfig", "fasolorn_model_spec",
-    "NuvezenConfig", "nuvezen_model_spec",
+    "NuvezenConfig", "nuvezen_model_spec", "ZugutarConfig", "zugutar_model_spec",
     "read_config_json", "architecture_of", "load_config",
 ]

@@ -59,12 +59,14 @@ class ScheduleEntry:
     ``layer`` indexes ``ModelSpec.layers`` (the weights that run).  ``cache``
     names the cache slot the mixer uses: entries with the same ``cache`` share
     keys and values.  ``writes_cache`` is false for an entry that only reads a
-    slot another entry filled earlier in the same step.
+    slot another entry filled earlier in the same step.  ``adds_embedding``: the
+    stream as it was before the first layer is added to it before this entry runs.
     """
 
     layer: int
     cache: int
     writes_cache: bool = True
+    adds_embedding: bool = False
 
 
 @dataclass(frozen=True)

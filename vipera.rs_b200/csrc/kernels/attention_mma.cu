@@ -381,10 +381,12 @@ __global__ void attention_combine_kernel(const float* __restrict__ partial_ml, c
                                          const int* __restrict__ positions, int window, int chunk,
                                          const int* __restrict__ entry_starts, int keep_first, int sink,
                                          const float* __restrict__ sink_values = nullptr,
-                                         const float* __restrict__ gate = nullptr, long long gate_stride = 0) {
+                                         const float* __restrict__ gate = nullptr, long long gate_stride = 0,
+                                         int gate_per_head = 0) {
   // KEPT instances also know a learned sink (`sink_values` [heads]: exp(sink_h) joins head h's sum
   // instead of one) and an output gate (`gate`: the row of the entry's token, at gate + token *
-  // gate_stride, holds [heads * D] 32-bit pre-activations whose sigmoid multiplies the output).
+  // gate_stride, holds [heads * D] 32-bit pre-activations whose sigmoid multiplies the output; with
+  // gate_per_head [heads] of them, one for all values of a head).
   // `slices` counts the window's splits; with kept first keys (keep_first > 0) each row has one
   // more place, the last, for the kept keys the window has left behind.  sink != 0: a key of score
   // 0 without a value joins the softmax, which adds exp2(-max) to the sum.
@@ -454,7 +456,7 @@ __global__ void attention_combine_kernel(const float* __restrict__ partial_ml, c
   }
   if (KEPT && sink) total += sink_values ? exp2f(sink_values[blockIdx.y] * 1.4426950408889634f - mine) : exp2f(-mine);   // the maxima are in units of log2
   float result = value / total;
-  if (KEPT && gate) result *= 1.0f / (1.0f + expf(-gate[out_token * gate_stride + static_cast<size_t>(blockIdx.y) * D + threadIdx.x]));
+  if (KEPT && gate) result *= 1.0f / (1.0f + expf(-gate[out_token * gate_stride + (gate_per_head ? static_cast<size_t>(blockIdx.y) : static_cast<size_t>(blockIdx.y) * D + threadIdx.x)]));
   if (WIDE) reinterpret_cast<float*>(out)[out_row * D + threadIdx.x] = result;
   else out[out_row * D + threadIdx.x] = __float2bfloat16_rn(result);
 }
@@ -494,7 +496,7 @@ attention_decode_cluster_kernel(const __nv_bfloat16* __restrict__ q, const __nv_
                                 const int* __restrict__ block_table, int table_width, int page_size, int page_shift,
                                 int num_heads, int num_kv_heads, float scale, int window, __nv_bfloat16* __restrict__ out,
                                 const float* __restrict__ sink_values, const float* __restrict__ gate,
-                                long long gate_stride) {
+                                long long gate_stride, int gate_per_head) {
   constexpr int kKeys = 32;
   constexpr int kWarpTile = 2 * kKeys * D * 2;  // bytes of one warp's key and value tiles
   constexpr int kRow = D + 4;                   // floats of a partial row: D outputs, max, sum, padding
@@ -667,7 +669,7 @@ attention_decode_cluster_kernel(const __nv_bfloat16* __restrict__ q, const __nv_
       const int head = kv_head * group + head_in_group;
       if (EXT && sink_values) total += exp2f(sink_values[head] * 1.4426950408889634f - best);   // the maxima are in units of log2
       float result = value / total;
-      if (EXT && gate) result *= 1.0f / (1.0f + expf(-gate[static_cast<size_t>(entry) * gate_stride + static_cast<size_t>(head) * D + col]));
+      if (EXT && gate) result *= 1.0f / (1.0f + expf(-gate[static_cast<size_t>(entry) * gate_stride + (gate_per_head ? static_cast<size_t>(head) : static_cast<size_t>(head) * D + col)]));
       out[(static_cast<size_t>(entry) * num_heads + head) * D + col] = __float2bfloat16_rn(result);
     }
   }
@@ -757,11 +759,12 @@ template <int D, int BLOCKS, bool PREFETCH, bool EXT = false>
 int launch_decode_cluster(const void* q, void* out, const void* k_pool, const void* v_pool, const int* positions,
                           const int* block_table, int table_width, int page_size, int page_shift, int num_entries,
                           int num_heads, int num_kv_heads, float scale, int window, cudaStream_t s,
-                          const float* sink_values = nullptr, const float* gate = nullptr, long long gate_stride = 0) {
+                          const float* sink_values = nullptr, const float* gate = nullptr, long long gate_stride = 0,
+                  int gate_per_head = 0) {
   if (!EXT && (sink_values || gate))
     return launch_decode_cluster<D, BLOCKS, PREFETCH, true>(q, out, k_pool, v_pool, positions, block_table, table_width,
                                                             page_size, page_shift, num_entries, num_heads, num_kv_heads,
-                                                            scale, window, s, sink_values, gate, gate_stride);
+                                                            scale, window, s, sink_values, gate, gate_stride, gate_per_head);
   constexpr int kSmem = 16 * D * 2 + 4 * (PREFETCH ? 2 : 1) * (2 * 32 * D * 2) + 16 * (D + 4) * 4;
   static int configured = 0;  // 1: ready, -1: this cluster size cannot be launched here
   if (configured == 0) {
@@ -795,7 +798,7 @@ int launch_decode_cluster(const void* q, void* out, const void* k_pool, const vo
                                          static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_pool),
                                          static_cast<const __nv_bfloat16*>(v_pool), positions, block_table, table_width,
                                          page_size, page_shift, num_heads, num_kv_heads, scale, window,
-                                         static_cast<__nv_bfloat16*>(out), sink_values, gate, gate_stride);
+                                         static_cast<__nv_bfloat16*>(out), sink_values, gate, gate_stride, gate_per_head);
   return error == cudaSuccess ? VIPERA_OK : static_cast<int>(error);
 }
 
@@ -804,7 +807,8 @@ int launch_decode(const void* q, void* out, const void* k_pool, const void* v_po
                   const int* block_table, int table_width, int page_size, int num_entries, int num_heads,
                   int num_kv_heads, float scale, int window, int chunk, int num_splits, float* partial_ml,
                   float* partial_out, const int* entry_starts, int keep_first, int sink, cudaStream_t s,
-                  const float* sink_values = nullptr, const float* gate = nullptr, long long gate_stride = 0) {
+                  const float* sink_values = nullptr, const float* gate = nullptr, long long gate_stride = 0,
+                  int gate_per_head = 0) {
   constexpr int kSmem = 16 * D * 2 + 4 * 2 * 32 * D * 2;
   int page_shift = -1;
   if ((page_size & (page_size - 1)) == 0) {
@@ -817,16 +821,16 @@ int launch_decode(const void* q, void* out, const void* k_pool, const void* v_po
                                              : cluster_decode_choice(num_entries, num_heads, num_kv_heads, chunk * num_splits);
   if (cluster.blocks == 8 && cluster.prefetch)
     return launch_decode_cluster<D, 8, true>(q, out, k_pool, v_pool, positions, block_table, table_width, page_size,
-                                             page_shift, num_entries, num_heads, num_kv_heads, scale, window, s, sink_values, gate, gate_stride);
+                                             page_shift, num_entries, num_heads, num_kv_heads, scale, window, s, sink_values, gate, gate_stride, gate_per_head);
   if (cluster.blocks == 8)
     return launch_decode_cluster<D, 8, false>(q, out, k_pool, v_pool, positions, block_table, table_width, page_size,
-                                              page_shift, num_entries, num_heads, num_kv_heads, scale, window, s, sink_values, gate, gate_stride);
+                                              page_shift, num_entries, num_heads, num_kv_heads, scale, window, s, sink_values, gate, gate_stride, gate_per_head);
   if (cluster.blocks == 16 && cluster.prefetch)
     return launch_decode_cluster<D, 16, true>(q, out, k_pool, v_pool, positions, block_table, table_width, page_size,
-                                              page_shift, num_entries, num_heads, num_kv_heads, scale, window, s, sink_values, gate, gate_stride);
+                                              page_shift, num_entries, num_heads, num_kv_heads, scale, window, s, sink_values, gate, gate_stride, gate_per_head);
   if (cluster.blocks == 16)
     return launch_decode_cluster<D, 16, false>(q, out, k_pool, v_pool, positions, block_table, table_width, page_size,
-                                               page_shift, num_entries, num_heads, num_kv_heads, scale, window, s, sink_values, gate, gate_stride);
+                                               page_shift, num_entries, num_heads, num_kv_heads, scale, window, s, sink_values, gate, gate_stride, gate_per_head);
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
@@ -845,7 +849,7 @@ int launch_decode(const void* q, void* out, const void* k_pool, const void* v_po
     return vipera_launch(attention_combine_kernel<D, true>, dim3(num_entries, num_heads), D, 0, s,
         static_cast<const float*>(partial_ml), static_cast<const float*>(partial_out), num_splits,
         static_cast<__nv_bfloat16*>(out), num_heads, positions, window, chunk, entry_starts, keep_first, sink,
-        sink_values, gate, gate_stride);
+        sink_values, gate, gate_stride, gate_per_head);
   }
   dim3 grid(num_entries, num_kv_heads, num_splits);
   int status = vipera_launch(attention_decode_kernel<D>, grid, 128, kSmem, s,
@@ -856,7 +860,7 @@ int launch_decode(const void* q, void* out, const void* k_pool, const void* v_po
   return vipera_launch(attention_combine_kernel<D>, dim3(num_entries, num_heads), D, 0, s,
       static_cast<const float*>(partial_ml), static_cast<const float*>(partial_out), num_splits,
       static_cast<__nv_bfloat16*>(out), num_heads, positions, window, chunk, entry_starts, 0, 0,
-      static_cast<const float*>(nullptr), static_cast<const float*>(nullptr), 0LL);
+      static_cast<const float*>(nullptr), static_cast<const float*>(nullptr), 0LL, 0);
 }
 
 // Single tokens, every query head against every KV head's values: out [entries, heads * kv_heads, D].
@@ -888,7 +892,7 @@ int launch_decode_pairs(const void* q, void* out, const void* k_pool, const void
   return vipera_launch(attention_combine_kernel<D, false, true>, dim3(num_entries, pairs), D, 0, s,
       static_cast<const float*>(partial_ml), static_cast<const float*>(partial_out), num_splits,
       static_cast<__nv_bfloat16*>(out), pairs, positions, 0, chunk, static_cast<const int*>(nullptr), 0, 0,
-      static_cast<const float*>(nullptr), static_cast<const float*>(nullptr), 0LL);
+      static_cast<const float*>(nullptr), static_cast<const float*>(nullptr), 0LL, 0);
 }
 
 }  // namespace
@@ -971,7 +975,8 @@ static int run_decode(const void* q, void* out, const void* k_pool, const void* 
                       const int* block_table, int table_width, int page_size, int num_entries, int num_heads,
                       int num_kv_heads, int head_dim, float scale, int window, int chunk, int num_splits, float* scratch,
                       size_t scratch_floats, const int* entry_starts, int keep_first, int sink, void* stream,
-                      const float* sink_values = nullptr, const float* gate = nullptr, long long gate_stride = 0) {
+                      const float* sink_values = nullptr, const float* gate = nullptr, long long gate_stride = 0,
+                  int gate_per_head = 0) {
   if (num_entries <= 0) return VIPERA_OK;
   if (sink_values) sink = 1;
   if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || keep_first < 0) return VIPERA_BAD_SHAPE;
@@ -988,11 +993,11 @@ static int run_decode(const void* q, void* out, const void* k_pool, const void* 
   if (head_dim == 128)
     return launch_decode<128>(q, out, k_pool, v_pool, positions, block_table, table_width, page_size, num_entries,
                               num_heads, num_kv_heads, scale, window, chunk, num_splits, partial_ml, partial_out,
-                              entry_starts, keep_first, sink, s, sink_values, gate, gate_stride);
+                              entry_starts, keep_first, sink, s, sink_values, gate, gate_stride, gate_per_head);
   if (head_dim == 64)
     return launch_decode<64>(q, out, k_pool, v_pool, positions, block_table, table_width, page_size, num_entries,
                              num_heads, num_kv_heads, scale, window, chunk, num_splits, partial_ml, partial_out,
-                             entry_starts, keep_first, sink, s, sink_values, gate, gate_stride);
+                             entry_starts, keep_first, sink, s, sink_values, gate, gate_stride, gate_per_head);
   return VIPERA_BAD_SHAPE;
 }
 
@@ -1049,17 +1054,18 @@ VIPERA_API int vipera_attention_decode_kept(const void* q, void* out, const void
 
 // The same with a learned sink per query head (`sink_values` [heads], null: the plain sink flag counts)
 // and an output gate (`gate`, null: none: 32-bit pre-activations, the row of token t at gate + t *
-// gate_stride holding [heads * d] values; t is the entry's index, or its token's with `entry_starts`).
+// gate_stride holding [heads * d] values, or [heads] with `gate_per_head`; t is the entry's index, or its token's
+// with `entry_starts`).
 VIPERA_API int vipera_attention_decode_gated(const void* q, void* out, const void* k_pool, const void* v_pool,
                                              const int* positions, const int* block_table, int table_width,
                                              int page_size, int num_entries, int num_heads, int num_kv_heads,
                                              int head_dim, float scale, int window, int chunk, int num_splits,
                                              float* scratch, size_t scratch_floats, const int* entry_starts,
                                              int keep_first, int sink, const float* sink_values, const float* gate,
-                                             long long gate_stride, void* stream) {
+                                             long long gate_stride, int gate_per_head, void* stream) {
   return run_decode(q, out, k_pool, v_pool, positions, block_table, table_width, page_size, num_entries, num_heads,
                     num_kv_heads, head_dim, scale, window, chunk, num_splits, scratch, scratch_floats, entry_starts,
-                    keep_first, sink, stream, sink_values, gate, gate_stride);
+                    keep_first, sink, stream, sink_values, gate, gate_stride, gate_per_head);
 }
 
 VIPERA_API const char* vipera_attention_mma_status_text(int status) { return vipera_status_text(status); }

@@ -76,10 +76,11 @@ struct Params {
   int* status;
   // Options of the ending.  sink_values [heads] (null: none): exp(sink_h) joins head h's denominator
   // (a learned sink: a term of the softmax sum that stands for no token; the score scale does not apply to it).  gate (null: none): the output is multiplied by
-  // sigmoid(gate[t * gate_stride + h * d + e]), a 32-bit pre-activation.
+  // sigmoid(gate[t * gate_stride + h * d + e]), a 32-bit pre-activation (gate_per_head: gate[t * gate_stride + h]).
   const float* sink_values;
   const float* gate;
   long long gate_stride;
+  int gate_per_head;
 };
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
@@ -514,7 +515,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap k_map, const __g
           joined[k] = own_has_tiles ? __uint_as_float(v[k]) * own_factor : 0.0f;
           if (other_has_tiles) joined[k] = fmaf(__uint_as_float(w[k]), other_factor, joined[k]);
         }
-        if (EXT && p.gate != nullptr && row < tokens_here) {
+        if (EXT && p.gate != nullptr && p.gate_per_head && row < tokens_here) {
+          const float z = p.gate[static_cast<size_t>(token0 + row) * p.gate_stride + head];
+          const float factor = 1.0f / (1.0f + __expf(-z));
+#pragma unroll
+          for (int k = 0; k < 32; ++k) joined[k] *= factor;
+        } else if (EXT && p.gate != nullptr && row < tokens_here) {
           const float4* gate_row = reinterpret_cast<const float4*>(
               p.gate + static_cast<size_t>(token0 + row) * p.gate_stride + static_cast<size_t>(head) * D + col0 + c);
 #pragma unroll
@@ -898,15 +904,16 @@ int launch_attention(const CUtensorMap& k_map, const CUtensorMap& v_map, const C
 // kernel ran out.
 // `sink_values` [heads] (null: none): a learned sink per query head; `gate` (null: none): 32-bit
 // pre-activations of an output gate, row t at gate + t * gate_stride, [heads * d] values (the base and
-// the stride whole multiples of four floats).
+// the stride whole multiples of four floats), or with `gate_per_head` [heads] values, one for a whole head.
 VIPERA_API int vipera_attention_prefill_tc_gated(const void* q, void* out, const void* k_pool, const void* v_pool,
                                                  const int* entry_starts, const int* entry_pos0, const int* block_table,
                                                  int table_width, int page_size, int num_entries, int num_tokens,
                                                  int num_heads, int num_kv_heads, int head_dim, float scale, int window,
                                                  int num_pages, int skip_single, const float* sink_values,
-                                                 const float* gate, long long gate_stride, int* status, void* stream) {
+                                                 const float* gate, long long gate_stride, int gate_per_head, int* status,
+                                                 void* stream) {
   if (num_tokens <= 0 || num_entries <= 0) return VIPERA_OK;
-  if (gate && ((reinterpret_cast<uintptr_t>(gate) & 15) || (gate_stride & 3))) return VIPERA_BAD_ARGUMENT;
+  if (gate && !gate_per_head && ((reinterpret_cast<uintptr_t>(gate) & 15) || (gate_stride & 3))) return VIPERA_BAD_ARGUMENT;
   if ((head_dim != 64 && head_dim != 128) || num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads || page_size <= 0 || num_pages <= 0)
     return VIPERA_BAD_SHAPE;
   if (!status) return VIPERA_BAD_ARGUMENT;
@@ -930,6 +937,7 @@ VIPERA_API int vipera_attention_prefill_tc_gated(const void* q, void* out, const
   p.sink_values = sink_values;
   p.gate = gate;
   p.gate_stride = gate_stride;
+  p.gate_per_head = gate_per_head;
   // at most one partly filled tile per entry beyond the full ones
   dim3 grid(num_heads, (num_tokens + kQ - 1) / kQ + num_entries);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -954,7 +962,7 @@ VIPERA_API int vipera_attention_prefill_tc(const void* q, void* out, const void*
                                            int num_pages, int skip_single, int* status, void* stream) {
   return vipera_attention_prefill_tc_gated(q, out, k_pool, v_pool, entry_starts, entry_pos0, block_table, table_width,
                                            page_size, num_entries, num_tokens, num_heads, num_kv_heads, head_dim, scale,
-                                           window, num_pages, skip_single, nullptr, nullptr, 0, status, stream);
+                                           window, num_pages, skip_single, nullptr, nullptr, 0, 0, status, stream);
 }
 
 VIPERA_API const char* vipera_attention_tc_status_text(int status) { return vipera_status_text(status); }

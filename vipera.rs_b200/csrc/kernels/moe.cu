@@ -37,6 +37,8 @@
 // `always_gate`: the router's matrix has one row more, and the always-used units' weight is the
 // sigmoid of that row's product with h.  ACT_CLAMPED: a gated unit with bounds (`unit_limit`, one per
 // unit with matrices) and the slope `unit_slope` inside its sigmoid.
+// `input_weight`: a chosen expert's weight multiplies what it reads, y_e = D_e (act(w_e G_e h) * (w_e U_e h)),
+// and not its output (the always-used units' weight stays on their output).
 #include "common.cuh"
 
 constexpr int kTileRows = 32;
@@ -76,7 +78,16 @@ struct MoeParams {
   int always_gate;          // 1: the always-used units' weight is sigmoid(the router's last row . h)
   const float* unit_limit;  // ACT_CLAMPED: [matrices]
   float unit_slope;
+  int input_weight;         // 1: a chosen expert's weight multiplies its input
 };
+
+// The weight of assignment `a` on the unit's input and on its output.
+__device__ __forceinline__ float moe_input_weight(const MoeParams& p, int a) {
+  return p.input_weight && a % p.slots < p.top ? p.weight[a] : 1.0f;
+}
+__device__ __forceinline__ float moe_output_weight(const MoeParams& p, int a) {
+  return p.input_weight && a % p.slots < p.top ? 1.0f : p.weight[a];
+}
 
 // The gated unit of matrix `unit`.
 __device__ __forceinline__ float moe_gated(const MoeParams& p, float gate, float up, int unit) {
@@ -324,6 +335,18 @@ moe_gather_kernel(MoeParams p) {
     return;
   }
   const uint4* src = reinterpret_cast<const uint4*>(static_cast<const T*>(p.h) + static_cast<size_t>(a / p.slots) * p.hidden);
+  if (p.input_weight && a % p.slots < p.top) {
+    constexpr int kPer = 16 / static_cast<int>(sizeof(T));
+    const float w = p.weight[a];
+    for (int i = threadIdx.x; i < vectors; i += blockDim.x) {
+      uint4 raw = src[i];
+      T* values = reinterpret_cast<T*>(&raw);
+#pragma unroll
+      for (int e = 0; e < kPer; ++e) values[e] = from_float<T>(w * to_float<T>(values[e]));
+      dst[i] = raw;
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < vectors; i += blockDim.x) dst[i] = src[i];
 }
 
@@ -337,7 +360,7 @@ moe_scatter_kernel(MoeParams p) {
   if (i >= static_cast<long long>(p.num_tokens) * p.slots * quarter) return;
   const int a = static_cast<int>(i / quarter), c = static_cast<int>(i % quarter);
   if (p.rank[a] < 0) return;   // the router's block wrote this row
-  const float w = p.weight[a];
+  const float w = moe_output_weight(p, a);
   float4 v = reinterpret_cast<const float4*>(p.ys + static_cast<size_t>(p.rank[a]) * p.hidden)[c];
   v.x *= w, v.y *= w, v.z *= w, v.w *= w;
   reinterpret_cast<float4*>(p.rows + static_cast<size_t>(a) * p.hidden)[c] = v;
@@ -440,20 +463,21 @@ moe_skinny_kernel(MoeParams p) {
 #pragma unroll
   for (int r = 0; r < kSkinnyRows; ++r) {
     if (r >= rows) continue;
+    const float w_in = FIRST && p.input_weight ? moe_input_weight(p, p.order[first + r]) : 1.0f;
     if (GATED) {
 #pragma unroll
       for (int f = 0; f < 2; ++f)
         if (col0 + f < outer)
           static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + col0 + f] =
-              from_float<T>(moe_gated(p, acc[2 * f][r], acc[2 * f + 1][r], expert));
+              from_float<T>(moe_gated(p, w_in * acc[2 * f][r], w_in * acc[2 * f + 1][r], expert));
     } else if (FIRST) {
 #pragma unroll
       for (int j = 0; j < 4; ++j)
         if (col0 + j < outer)
-          static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + col0 + j] = from_float<T>(gate_activation(acc[j][r], p.activation));
+          static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + col0 + j] = from_float<T>(gate_activation(w_in * acc[j][r], p.activation));
     } else {
       const int a = p.order[first + r];
-      const float weight = p.weight[a];
+      const float weight = moe_output_weight(p, a);
 #pragma unroll
       for (int j = 0; j < 4; ++j)
         if (col0 + j < outer) p.rows[static_cast<size_t>(a) * p.hidden + col0 + j] = weight * acc[j][r];
@@ -534,18 +558,19 @@ moe_product_kernel(MoeParams p) {
   for (int i = 0; i < 2; ++i) {
     const int r = ty + 16 * i;
     if (r >= rows) continue;
+    const float w_in = FIRST && p.input_weight ? moe_input_weight(p, p.order[first + r]) : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int c = col0 + tx + 16 * j;
       if (c >= outer) continue;
       if (GATED) {
         static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + c] =
-            from_float<T>(moe_gated(p, acc0[i][j], acc1[i][j], expert));
+            from_float<T>(moe_gated(p, w_in * acc0[i][j], w_in * acc1[i][j], expert));
       } else if (FIRST) {
-        static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + c] = from_float<T>(gate_activation(acc0[i][j], p.activation));
+        static_cast<T*>(p.act)[static_cast<size_t>(first + r) * p.ff + c] = from_float<T>(gate_activation(w_in * acc0[i][j], p.activation));
       } else {
         const int a = p.order[first + r];
-        p.rows[static_cast<size_t>(a) * p.hidden + c] = p.weight[a] * acc0[i][j];
+        p.rows[static_cast<size_t>(a) * p.hidden + c] = moe_output_weight(p, a) * acc0[i][j];
       }
     }
   }

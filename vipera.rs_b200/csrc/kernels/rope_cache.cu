@@ -330,6 +330,131 @@ VIPERA_API int vipera_qk_prepare(const float* qkv, void* q_out, int dtype, int n
   return VIPERA_BAD_DTYPE;
 }
 
+// ---------------------------------------------------------------------------------------
+// The form with options per head.  Each query and key head is divided by its own root mean square,
+// sqrt(mean(x^2) + eps), and multiplied by a weight per value that all heads share (`q_norm`, `k_norm`
+// [head_dim]; null: left as it is); then its first `rot_dims` values turn; then a query is multiplied by a
+// number of its position (`q_factor` [positions], null: 1).  A warp per head of a token, eight to a block;
+// the head waits in shared memory, since a value's partner of the rotation belongs to another lane.
+// Rows of the input may hold more than q, k and v (`row_stride` values apart).
+// ---------------------------------------------------------------------------------------
+constexpr int kHeadWarps = 8;
+constexpr int kHeadMost = 256;   // values of a head
+
+struct HeadRowsParams {
+  const float* qkv;         // [tokens, row_stride]: q heads, k heads, v heads, and what else the product holds
+  long long row_stride;
+  void* q_out;              // [tokens, heads, head_dim]
+  int num_tokens, num_heads, num_kv_heads, head_dim, value_dim, rot_dims, style;
+  const float* q_norm;
+  const float* k_norm;
+  float eps;
+  const float* q_factor;
+  const int* positions;
+  const float* cos_table;   // [positions, rot_dims / 2]
+  const float* sin_table;
+  void* k_pool;
+  void* v_pool;
+  const int* token_entry;
+  const int* block_table;
+  int table_width, page_size, write_cache;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kHeadWarps * 32)
+head_rows_kernel(const HeadRowsParams p) {
+  __shared__ float rows[kHeadWarps][kHeadMost];
+  constexpr int kPerLane = kHeadMost / 32;
+  pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x;
+  const int job = blockIdx.y * kHeadWarps + warp;   // query heads, key heads, value heads
+  if (job >= p.num_heads + 2 * p.num_kv_heads) return;
+  const bool is_q = job < p.num_heads, is_v = job >= p.num_heads + p.num_kv_heads;
+  const int size = is_v ? p.value_dim : p.head_dim;
+  const int kv = is_v ? job - p.num_heads - p.num_kv_heads : job - p.num_heads;
+  // the step's description, the tables and the weights were there before the kernel ahead
+  const int position = p.positions[t];
+  const float* gain = is_v ? nullptr : (is_q ? p.q_norm : p.k_norm);
+  const float factor = is_q && p.q_factor ? p.q_factor[position] : 1.0f;
+  T* dst = nullptr;
+  if (is_q) {
+    dst = static_cast<T*>(p.q_out) + (static_cast<size_t>(t) * p.num_heads + job) * p.head_dim;
+  } else if (p.write_cache) {
+    const int page = p.block_table[static_cast<size_t>(p.token_entry[t]) * p.table_width + position / p.page_size];
+    if (page >= 0) {
+      const size_t at = static_cast<size_t>(page) * p.page_size + position % p.page_size;
+      dst = static_cast<T*>(is_v ? p.v_pool : p.k_pool) + (at * p.num_kv_heads + kv) * size;
+    }
+  }
+  const long long start = is_v ? static_cast<long long>(p.num_heads + p.num_kv_heads) * p.head_dim + static_cast<long long>(kv) * p.value_dim
+                               : static_cast<long long>(job) * p.head_dim;
+  const float* src = p.qkv + static_cast<long long>(t) * p.row_stride + start;
+  pdl_wait();
+  if (!dst) return;
+  float x[kPerLane];
+  float sum = 0.0f;
+#pragma unroll
+  for (int j = 0; j < kPerLane; ++j) {
+    const int e = lane + 32 * j;
+    x[j] = e < size ? src[e] : 0.0f;
+    sum = fmaf(x[j], x[j], sum);
+  }
+  if (gain) {
+    const float inverse = 1.0f / sqrtf(warp_sum(sum) / static_cast<float>(size) + p.eps);
+#pragma unroll
+    for (int j = 0; j < kPerLane; ++j) {
+      const int e = lane + 32 * j;
+      if (e < size) x[j] = x[j] * inverse * gain[e];
+    }
+  }
+  if (!is_v && p.style != ROPE_NONE && p.rot_dims > 0) {
+    const int half = p.rot_dims >> 1;
+    const float* cos_row = p.cos_table + static_cast<size_t>(position) * half;
+    const float* sin_row = p.sin_table + static_cast<size_t>(position) * half;
+    float* row = rows[warp];
+#pragma unroll
+    for (int j = 0; j < kPerLane; ++j)
+      if (lane + 32 * j < p.rot_dims) row[lane + 32 * j] = x[j];
+    __syncwarp();
+#pragma unroll
+    for (int j = 0; j < kPerLane; ++j) {
+      const int e = lane + 32 * j;
+      if (e < p.rot_dims) {
+        const bool second = p.style == ROPE_INTERLEAVED ? (e & 1) : e >= half;
+        const int i = p.style == ROPE_INTERLEAVED ? e >> 1 : (second ? e - half : e);
+        const float partner = row[p.style == ROPE_INTERLEAVED ? (e ^ 1) : (second ? e - half : e + half)];
+        const float c = cos_row[i], s = sin_row[i];
+        x[j] = second ? fmaf(partner, s, x[j] * c) : fmaf(-partner, s, x[j] * c);
+      }
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < kPerLane; ++j) {
+    const int e = lane + 32 * j;
+    if (e < size) dst[e] = from_float<T>(x[j] * factor);
+  }
+}
+
+// dtype: the type of q_out and of the pools.
+VIPERA_API int vipera_head_rows(const HeadRowsParams* params, int dtype, void* stream) {
+  const HeadRowsParams& p = *params;
+  if (p.num_tokens <= 0) return VIPERA_OK;
+  if (p.head_dim <= 0 || p.head_dim > kHeadMost || p.value_dim <= 0 || p.value_dim > kHeadMost || p.num_heads <= 0 ||
+      p.num_kv_heads <= 0 || p.rot_dims < 0 || (p.rot_dims & 1) || p.rot_dims > p.head_dim)
+    return VIPERA_BAD_SHAPE;
+  if (!p.qkv || !p.q_out || !p.positions) return VIPERA_BAD_ARGUMENT;
+  if (p.style != ROPE_NONE && p.rot_dims > 0 && (!p.cos_table || !p.sin_table)) return VIPERA_BAD_ARGUMENT;
+  if (p.write_cache && (!p.k_pool || !p.v_pool || !p.token_entry || !p.block_table || p.page_size <= 0)) return VIPERA_BAD_ARGUMENT;
+  const dim3 grid(p.num_tokens, (p.num_heads + 2 * p.num_kv_heads + kHeadWarps - 1) / kHeadWarps);
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (dtype == VIPERA_F32) return vipera_launch(head_rows_kernel<float>, grid, kHeadWarps * 32, 0, s, p);
+  if (dtype == VIPERA_BF16) return vipera_launch(head_rows_kernel<__nv_bfloat16>, grid, kHeadWarps * 32, 0, s, p);
+  return VIPERA_BAD_DTYPE;
+}
+
+VIPERA_API int vipera_head_rows_params_size() { return static_cast<int>(sizeof(HeadRowsParams)); }
+
 VIPERA_API int vipera_rope_cache(const float* qkv, void* q_out, int dtype, int num_tokens, int num_heads,
                                  int num_kv_heads, int head_dim, const int* positions,
                                  const float* cos_table, const float* sin_table, int style, void* k_pool,

@@ -13,7 +13,7 @@
 // ---------------------------------------------------------------------------------------
 template <typename TW>
 __global__ void embed_kernel(const TW* __restrict__ table, const int* __restrict__ tokens,
-                             float* __restrict__ out, int hidden, int vocab, float scale) {
+                             float* __restrict__ out, float* __restrict__ also, int hidden, int vocab, float scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -23,19 +23,25 @@ __global__ void embed_kernel(const TW* __restrict__ table, const int* __restrict
   token = min(max(token, 0), vocab - 1);
   const TW* row = table + static_cast<size_t>(token) * hidden;
   float* dst = out + static_cast<size_t>(t) * hidden;
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = scale * to_float<TW>(row[i]);
+  float* second = also ? also + static_cast<size_t>(t) * hidden : nullptr;
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+    const float value = scale * to_float<TW>(row[i]);
+    dst[i] = value;
+    if (second) second[i] = value;
+  }
 }
 
-VIPERA_API int vipera_embed(const void* table, int table_dtype, const int* tokens, float* out,
+// `also` (null: none): a second buffer that receives the same rows.
+VIPERA_API int vipera_embed(const void* table, int table_dtype, const int* tokens, float* out, float* also,
                             int num_tokens, int hidden, int vocab, float scale, void* stream) {
   if (num_tokens <= 0) return VIPERA_OK;
   if (hidden <= 0 || vocab <= 0) return VIPERA_BAD_SHAPE;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int threads = hidden >= 1024 ? 256 : 128;
   if (table_dtype == VIPERA_F32)
-    return vipera_launch(embed_kernel<float>, num_tokens, threads, 0, s, static_cast<const float*>(table), tokens, out, hidden, vocab, scale);
+    return vipera_launch(embed_kernel<float>, num_tokens, threads, 0, s, static_cast<const float*>(table), tokens, out, also, hidden, vocab, scale);
   if (table_dtype == VIPERA_BF16)
-    return vipera_launch(embed_kernel<__nv_bfloat16>, num_tokens, threads, 0, s, static_cast<const __nv_bfloat16*>(table), tokens, out, hidden, vocab, scale);
+    return vipera_launch(embed_kernel<__nv_bfloat16>, num_tokens, threads, 0, s, static_cast<const __nv_bfloat16*>(table), tokens, out, also, hidden, vocab, scale);
   return VIPERA_BAD_DTYPE;
 }
 
@@ -287,11 +293,16 @@ VIPERA_API const char* vipera_rowwise_status_text(int status) { return vipera_st
 // channel or null; either branch and either norm may be missing.  With `rows` the kernel computes
 // norms of the rows named there and leaves x as it is.  A block per row; VEC values to an access; the
 // row stays in registers between its passes where it is short enough.
+// A second form (join_normed_kernel) takes up to four branches, of which the first two may be divided
+// by the root mean square of their own row before they join (`normed`, `eps`; the norm's weight is in
+// `scale`):   x += scale_0 * b_0 / rms(b_0) + scale_1 * b_1 / rms(b_1) + scale_2 * b_2 + scale_3 * b_3
 // ---------------------------------------------------------------------------------------
 struct JoinBranch {
   const float* values;   // null: no such branch
   const float* scale;    // [hidden] or null: 1
   int parts;
+  int normed;            // 1: the branch's row is divided by sqrt(mean of its squares + eps)
+  float eps;
 };
 struct JoinNorm {
   const float* gain;     // null: no such norm
@@ -301,7 +312,7 @@ struct JoinNorm {
 struct JoinParams {
   float* x;
   const int* rows;
-  JoinBranch branch[2];
+  JoinBranch branch[4];
   JoinNorm norm[2];
   int num_rows, hidden, out_dtype;
 };
@@ -414,8 +425,146 @@ join_norms_kernel(const JoinParams p) {
   }
 }
 
+// The sum of a branch's parts for values i .. i + VEC - 1 of a row.
+template <int VEC>
+__device__ __forceinline__ JoinVector<VEC> join_parts(const JoinBranch& b, size_t row, int hidden, int i) {
+  JoinVector<VEC> sum;
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) sum.v[e] = 0.0f;
+  if (!b.values) return sum;
+  const float* src = b.values + row * b.parts * hidden + i;
+  sum = join_load<VEC>(src);
+  for (int part = 1; part < b.parts; ++part) {
+    const JoinVector<VEC> more = join_load<VEC>(src + static_cast<size_t>(part) * hidden);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) sum.v[e] += more.v[e];
+  }
+  return sum;
+}
+
+// Both sums over the block of kNormThreads threads, in one exchange.
+__device__ __forceinline__ float2 block_sum_pair(float a, float b, float2* scratch) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  a = warp_sum(a), b = warp_sum(b);
+  if (lane == 0) scratch[warp] = make_float2(a, b);
+  __syncthreads();
+  const float2 mine = lane < kNormThreads / 32 ? scratch[lane] : make_float2(0.0f, 0.0f);
+  return make_float2(warp_sum(mine.x), warp_sum(mine.y));
+}
+
+template <typename TO, int VEC>
+__global__ void __launch_bounds__(kNormThreads)
+join_normed_kernel(const JoinParams p) {
+  __shared__ float scratch[32];
+  __shared__ float2 pairs[kNormThreads / 32];
+  constexpr int kKept = VEC == 4 ? 4 : 8;
+  pdl_launch_dependents();
+  const int r = blockIdx.x;
+  const int first = threadIdx.x * VEC, step = kNormThreads * VEC;
+  const bool fits = p.hidden <= kKept * step;
+  pdl_wait();
+  const size_t row = p.rows ? p.rows[r] : r;
+  float* x = p.x + row * p.hidden;
+  const bool writes = p.rows == nullptr;
+  JoinVector<VEC> kept[kKept], own0[kKept], own1[kKept];
+  float squares0 = 0.0f, squares1 = 0.0f;
+  auto square = [](float& sum, const JoinVector<VEC>& v) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) sum = fmaf(v.v[e], v.v[e], sum);
+  };
+  if (fits) {
+    // the row of the stream with the plain branches, and the two branches that may be normed: all asked for together
+#pragma unroll
+    for (int j = 0; j < kKept; ++j) {
+      const int i = first + j * step;
+      if (i < p.hidden) {
+        own0[j] = join_parts<VEC>(p.branch[0], row, p.hidden, i);
+        own1[j] = join_parts<VEC>(p.branch[1], row, p.hidden, i);
+        kept[j] = join_load<VEC>(x + i);
+        join_add<VEC>(kept[j], p.branch[2], row, p.hidden, i);
+        join_add<VEC>(kept[j], p.branch[3], row, p.hidden, i);
+        square(squares0, own0[j]);
+        square(squares1, own1[j]);
+      }
+    }
+  } else {
+    for (int i = first; i < p.hidden; i += step) {
+      square(squares0, join_parts<VEC>(p.branch[0], row, p.hidden, i));
+      square(squares1, join_parts<VEC>(p.branch[1], row, p.hidden, i));
+    }
+  }
+  const float2 sums = block_sum_pair(squares0, squares1, pairs);
+  const float width = static_cast<float>(p.hidden);
+  const float inverse0 = p.branch[0].normed ? 1.0f / sqrtf(sums.x / width + p.branch[0].eps) : 1.0f;
+  const float inverse1 = p.branch[1].normed ? 1.0f / sqrtf(sums.y / width + p.branch[1].eps) : 1.0f;
+  auto add_scaled = [&](JoinVector<VEC>& to, const JoinVector<VEC>& own, const JoinBranch& b, float inverse, int i) {
+    if (!b.values) return;
+    JoinVector<VEC> s;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) s.v[e] = 1.0f;
+    if (b.scale) s = join_load<VEC>(b.scale + i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) to.v[e] = fmaf(s.v[e], own.v[e] * inverse, to.v[e]);
+  };
+  float squares = 0.0f;
+  auto joined = [&](int i) {   // rows too long for the registers
+    JoinVector<VEC> v = join_load<VEC>(x + i);
+    join_add<VEC>(v, p.branch[2], row, p.hidden, i);
+    join_add<VEC>(v, p.branch[3], row, p.hidden, i);
+    add_scaled(v, join_parts<VEC>(p.branch[0], row, p.hidden, i), p.branch[0], inverse0, i);
+    add_scaled(v, join_parts<VEC>(p.branch[1], row, p.hidden, i), p.branch[1], inverse1, i);
+    return v;
+  };
+  if (fits) {
+#pragma unroll
+    for (int j = 0; j < kKept; ++j) {
+      const int i = first + j * step;
+      if (i < p.hidden) {
+        add_scaled(kept[j], own0[j], p.branch[0], inverse0, i);
+        add_scaled(kept[j], own1[j], p.branch[1], inverse1, i);
+        square(squares, kept[j]);
+        if (writes) join_store<float, VEC>(x + i, kept[j]);
+      }
+    }
+  } else {
+    for (int i = first; i < p.hidden; i += step) {
+      const JoinVector<VEC> v = joined(i);
+      square(squares, v);
+      if (writes) join_store<float, VEC>(x + i, v);
+    }
+  }
+  if (!p.norm[0].gain && !p.norm[1].gain) return;
+  const float mean = block_sum(squares, scratch) / width;
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    const JoinNorm& norm = p.norm[n];
+    if (!norm.gain) continue;
+    const float inverse = 1.0f / sqrtf(mean + norm.eps);
+    TO* out = static_cast<TO*>(norm.out) + static_cast<size_t>(r) * p.hidden;
+    auto finish = [&](JoinVector<VEC> v, int i) {
+      const JoinVector<VEC> g = join_load<VEC>(norm.gain + i);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v.v[e] = v.v[e] * inverse * g.v[e];
+      join_store<TO, VEC>(out + i, v);
+    };
+    if (fits) {
+#pragma unroll
+      for (int j = 0; j < kKept; ++j) {
+        const int i = first + j * step;
+        if (i < p.hidden) finish(kept[j], i);
+      }
+    } else {
+      for (int i = first; i < p.hidden; i += step) finish(writes ? join_load<VEC>(x + i) : joined(i), i);
+    }
+  }
+}
+
 template <typename TO>
 static int launch_join(const JoinParams& p, bool vectors, cudaStream_t s) {
+  if (p.branch[2].values || p.branch[3].values || p.branch[0].normed || p.branch[1].normed) {
+    if (vectors) return vipera_launch(join_normed_kernel<TO, 4>, p.num_rows, kNormThreads, 0, s, p);
+    return vipera_launch(join_normed_kernel<TO, 1>, p.num_rows, kNormThreads, 0, s, p);
+  }
   if (vectors) return vipera_launch(join_norms_kernel<TO, 4>, p.num_rows, kNormThreads, 0, s, p);
   return vipera_launch(join_norms_kernel<TO, 1>, p.num_rows, kNormThreads, 0, s, p);
 }
@@ -426,11 +575,14 @@ VIPERA_API int vipera_join_norms(const JoinParams* params, void* stream) {
   if (p.num_rows <= 0) return VIPERA_OK;
   if (p.hidden <= 0 || !p.x) return VIPERA_BAD_SHAPE;
   uintptr_t bases = reinterpret_cast<uintptr_t>(p.x);
-  for (int i = 0; i < 2; ++i) {
+  for (int i = 0; i < 4; ++i) {
     if (p.branch[i].values && p.branch[i].parts <= 0) return VIPERA_BAD_ARGUMENT;
+    if (p.branch[i].normed && (i > 1 || !p.branch[i].values)) return VIPERA_BAD_ARGUMENT;
+    bases |= reinterpret_cast<uintptr_t>(p.branch[i].values) | reinterpret_cast<uintptr_t>(p.branch[i].scale);
+  }
+  for (int i = 0; i < 2; ++i) {
     if (p.norm[i].gain && !p.norm[i].out) return VIPERA_BAD_ARGUMENT;
-    bases |= reinterpret_cast<uintptr_t>(p.branch[i].values) | reinterpret_cast<uintptr_t>(p.branch[i].scale) |
-             reinterpret_cast<uintptr_t>(p.norm[i].gain) | reinterpret_cast<uintptr_t>(p.norm[i].out);
+    bases |= reinterpret_cast<uintptr_t>(p.norm[i].gain) | reinterpret_cast<uintptr_t>(p.norm[i].out);
   }
   const bool vectors = p.hidden % 4 == 0 && (bases & 15) == 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

@@ -81,11 +81,12 @@ def kv_bytes_per_token(spec: ModelSpec, element_bytes: int) -> int:
 
 
 def workspace_bytes(spec: ModelSpec, batch: int, element_bytes: int, tokens: int = PLANNED_STEP_TOKENS) -> int:
-    """The 32-bit residual stream, the normalised input, the most any layer asks for (layers
+    """The 32-bit residual stream (twice where the embedding's rows are kept beside it), the normalised input, the most any layer asks for (layers
     share their buffers), the products' scratch for partial sums, and the 32-bit logits rows of
     a batch."""
     layers = max(BLOCKS.find(layer.block).workspace_bytes(layer, tokens, element_bytes) for layer in spec.layers)
-    return (tokens * spec.hidden_size * (4 + element_bytes) + layers + PRODUCT_SCRATCH_BYTES
+    stream = 8 if any(entry.adds_embedding for entry in spec.schedule) else 4
+    return (tokens * spec.hidden_size * (stream + element_bytes) + layers + PRODUCT_SCRATCH_BYTES
             + batch * spec.vocab_size * 4)
 
 

@@ -21,7 +21,7 @@ from .runner import ModelRunner, StepInput
 
 class Replayer:
     def __init__(self, model_dir: str, dtype: str, *, max_tokens: int, page_size: int = 64,
-                 device: str = "cuda:0", max_live: int = 8):
+                 device: str = "cuda:0", max_live: int = 4):
         self.model = load_model(model_dir, dtype, device)
         pages = max(1, (int(max_tokens) + page_size - 1) // page_size)
         self.pools = CachePools(self.model.cache_requests, page_size=page_size, num_pages=pages,

@@ -95,7 +95,7 @@ class KernelProfile:
         "gemm_tc": "proj", "gemm_tc_rope": "proj", "gemv_small": "proj", "gemm_simt": "proj",
         "attention": "attention", "attention_prefill": "attention", "attention_prefill_tc": "attention",
         "attention_decode": "attention", "mlstm": "recurrence", "mamba_scan": "recurrence", "gla": "recurrence",
-        "lightning": "recurrence", "moe": "experts",
+        "lightning": "recurrence", "mamba2": "recurrence", "moe": "experts",
         "layernorm": "norm", "causal_conv": "conv",
         "argmax": "sample", "sample": "sample", "apply_penalties": "sample", "feed_tokens": "sample",
         "logprobs": "sample",
@@ -193,15 +193,16 @@ def _opt(tensor: Optional[torch.Tensor], name: str, dtype=None):
 
 
 # ----------------------------------------------------------------------------------------
-def embed(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
-    """out[t, :] = scale * table[tokens[t], :] as float32."""
+def embed(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, scale: float = 1.0,
+          also: Optional[torch.Tensor] = None) -> None:
+    """out[t, :] = scale * table[tokens[t], :] as float32; ``also`` receives the same rows."""
     fn = _function("rowwise", "vipera_embed",
-                   [_c_void, _c_int, _c_void, _c_void, _c_int, _c_int, _c_int, _c_float, _c_void])
+                   [_c_void, _c_int, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_float, _c_void])
     count, hidden = out.shape
-    if table.shape[1] != hidden or tokens.numel() != count:
+    if table.shape[1] != hidden or tokens.numel() != count or (also is not None and also.shape != out.shape):
         raise InvalidArgumentError("embed: shapes of table, tokens and out do not agree")
     _check(fn(_gpu(table, "table"), dtype_code(table.dtype), _gpu(tokens, "tokens", torch.int32),
-              _gpu(out, "out", torch.float32), count, hidden, table.shape[0], float(scale), _stream()), "embed")
+              _gpu(out, "out", torch.float32), _opt(also, "also", torch.float32), count, hidden, table.shape[0], float(scale), _stream()), "embed")
 
 
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float,
@@ -235,7 +236,7 @@ def sm_count(device) -> int:
 
 
 class _JoinBranch(ctypes.Structure):
-    _fields_ = [("values", _c_void), ("scale", _c_void), ("parts", _c_int)]
+    _fields_ = [("values", _c_void), ("scale", _c_void), ("parts", _c_int), ("normed", _c_int), ("eps", _c_float)]
 
 
 class _JoinNorm(ctypes.Structure):
@@ -243,25 +244,35 @@ class _JoinNorm(ctypes.Structure):
 
 
 class _JoinParams(ctypes.Structure):
-    _fields_ = [("x", _c_void), ("rows", _c_void), ("branch", _JoinBranch * 2), ("norm", _JoinNorm * 2),
+    _fields_ = [("x", _c_void), ("rows", _c_void), ("branch", _JoinBranch * 4), ("norm", _JoinNorm * 2),
                 ("num_rows", _c_int), ("hidden", _c_int), ("out_dtype", _c_int)]
 
 
 def join_norms(x: torch.Tensor, branches=(), norms=(), rows: Optional[torch.Tensor] = None) -> None:
-    """Up to two branches join the float32 stream ``x`` [rows, hidden] and up to two RMS norms read the
+    """Up to four branches join the float32 stream ``x`` [rows, hidden] and up to two RMS norms read the
     result.  A branch is ``(values, parts, scale)``: ``x += scale * sum over the parts`` with values float32
-    [rows, parts * hidden] and scale float32 [hidden] or None.  A norm is ``(gain, eps, out)``.  With
-    ``rows`` (int32) the norms are those of the rows named there, and x stays as it is."""
+    [rows, parts * hidden] and scale float32 [hidden] or None; or ``(values, parts, scale, eps)``, for at most
+    two of them: the sum over the parts is first divided by its root mean square over the row.  A norm is
+    ``(gain, eps, out)``.  With ``rows`` (int32) the norms are those of the rows named there, and x stays as it
+    is."""
     fn = _function("rowwise", "vipera_join_norms", [ctypes.POINTER(_JoinParams), _c_void])
     _check_struct("rowwise", "vipera_join_params_size", _JoinParams)
     hidden = x.shape[-1]
     count = x.numel() // hidden if rows is None else rows.numel()
-    if len(branches) > 2 or len(norms) > 2 or not (branches or norms) or (rows is not None and not norms):
-        raise InvalidArgumentError("join_norms: up to two branches and up to two norms, at least one of them")
+    normed = [b for b in branches if len(b) > 3 and b[3] is not None]
+    plain = [b for b in branches if not (len(b) > 3 and b[3] is not None)]
+    if len(branches) > 4 or len(normed) > 2 or len(norms) > 2 or not (branches or norms) or (rows is not None and not norms):
+        raise InvalidArgumentError("join_norms: up to four branches, two of them normed, and up to two norms, at least one of them")
     p = _JoinParams()
     p.x, p.rows = _gpu(x, "x", torch.float32), _opt(rows, "rows", torch.int32)
     p.num_rows, p.hidden = count, hidden
-    for slot, (values, parts, scale) in zip(p.branch, branches):
+    # the normed branches have the first two places; the others fill what is left
+    order = [(0, b) for b in normed[:1]] + [(1, b) for b in normed[1:]]
+    order += list(zip(range(len(normed), 4), plain))
+    for place, branch in order:
+        slot, (values, parts, scale) = p.branch[place], branch[:3]
+        if len(branch) > 3 and branch[3] is not None:
+            slot.normed, slot.eps = 1, float(branch[3])
         if values.numel() != x.numel() * int(parts) or (scale is not None and scale.numel() != hidden):
             raise InvalidArgumentError("join_norms: a branch holds parts rows of the stream's width per row, its scale one "
                                        "number per channel")
@@ -393,6 +404,62 @@ def rope_cache_blend(qkv: torch.Tensor, q_out: torch.Tensor, *, num_heads: int, 
               _opt(blend, "blend", torch.float32), _stream()), "rope_cache")
 
 
+class _HeadRowsParams(ctypes.Structure):
+    _fields_ = [
+        ("qkv", _c_void), ("row_stride", ctypes.c_longlong), ("q_out", _c_void),
+        ("num_tokens", _c_int), ("num_heads", _c_int), ("num_kv_heads", _c_int), ("head_dim", _c_int), ("value_dim", _c_int),
+        ("rot_dims", _c_int), ("style", _c_int), ("q_norm", _c_void), ("k_norm", _c_void), ("eps", _c_float),
+        ("q_factor", _c_void), ("positions", _c_void), ("cos_table", _c_void), ("sin_table", _c_void),
+        ("k_pool", _c_void), ("v_pool", _c_void), ("token_entry", _c_void), ("block_table", _c_void),
+        ("table_width", _c_int), ("page_size", _c_int), ("write_cache", _c_int),
+    ]
+
+
+def head_rows(qkv: torch.Tensor, q_out: torch.Tensor, *, num_heads: int, num_kv_heads: int, head_dim: int,
+              value_dim: int, rot_dims: int, positions: torch.Tensor, cos: Optional[torch.Tensor],
+              sin: Optional[torch.Tensor], style: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
+              token_entry: torch.Tensor, block_table: torch.Tensor, page_size: int, write_cache: bool,
+              q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None, eps: float = 0.0,
+              q_factor: Optional[torch.Tensor] = None) -> None:
+    """Heads of a float32 product [tokens, >= (heads + kv_heads) * d + kv_heads * value_dim] on their way to q_out
+    [tokens, heads * d] and the cache: an RMS norm per head (``q_norm``, ``k_norm`` float32 [d], shared by all
+    heads, or None), rotation of a head's first ``rot_dims`` values, queries times ``q_factor[position]``."""
+    fn = _function("rope_cache", "vipera_head_rows", [ctypes.POINTER(_HeadRowsParams), _c_int, _c_void])
+    _check_struct("rope_cache", "vipera_head_rows_params_size", _HeadRowsParams)
+    count = qkv.shape[0]
+    if qkv.dim() != 2 or qkv.stride(1) != 1 or qkv.shape[1] < (num_heads + num_kv_heads) * head_dim + num_kv_heads * value_dim:
+        raise InvalidArgumentError("head_rows: qkv rows are too short for the head counts and sizes")
+    if tuple(q_out.shape) != (count, num_heads * head_dim) or positions.numel() < count or token_entry.numel() < count:
+        raise InvalidArgumentError("head_rows: q_out, positions or token_entry has the wrong shape")
+    if head_dim > 256 or value_dim > 256:
+        raise UnsupportedError("head_rows: heads of up to 256 values")
+    if rot_dims % 2 or not 0 <= rot_dims <= head_dim:
+        raise InvalidArgumentError("head_rows: the rotated values must be an even count within the head")
+    if style != ROPE_NONE and rot_dims:
+        if cos is None or sin is None or cos.shape[1] != rot_dims // 2 or sin.shape != cos.shape:
+            raise InvalidArgumentError("head_rows: cos/sin tables of width rot_dims/2 are needed")
+    for norm in (q_norm, k_norm):
+        if norm is not None and norm.numel() != head_dim:
+            raise InvalidArgumentError("head_rows: a norm per head has a weight per value of a head")
+    if write_cache and (k_pool.dtype != q_out.dtype or v_pool.dtype != q_out.dtype or
+                        k_pool.shape[1:] != (page_size, num_kv_heads, head_dim) or
+                        v_pool.shape[1:] != (page_size, num_kv_heads, value_dim)):
+        raise InvalidArgumentError("head_rows: cache pools must be [pages, page_size, kv_heads, d] and "
+                                   "[pages, page_size, kv_heads, value size] of the activation dtype")
+    p = _HeadRowsParams()
+    p.qkv, p.row_stride, p.q_out = _gpu(qkv, "qkv", torch.float32), int(qkv.stride(0)), _gpu(q_out, "q_out")
+    p.num_tokens, p.num_heads, p.num_kv_heads = int(count), int(num_heads), int(num_kv_heads)
+    p.head_dim, p.value_dim, p.rot_dims, p.style = int(head_dim), int(value_dim), int(rot_dims), int(style)
+    p.q_norm, p.k_norm, p.eps = _opt(q_norm, "q_norm", torch.float32), _opt(k_norm, "k_norm", torch.float32), float(eps)
+    p.q_factor, p.positions = _opt(q_factor, "q_factor", torch.float32), _gpu(positions, "positions", torch.int32)
+    p.cos_table, p.sin_table = _opt(cos, "cos", torch.float32), _opt(sin, "sin", torch.float32)
+    p.k_pool, p.v_pool = _gpu(k_pool, "k_pool"), _gpu(v_pool, "v_pool")
+    p.token_entry = _gpu(token_entry, "token_entry", torch.int32)
+    p.block_table, p.table_width = _gpu(block_table, "block_table", torch.int32), int(block_table.shape[1])
+    p.page_size, p.write_cache = int(page_size), 1 if write_cache else 0
+    _check(fn(ctypes.byref(p), dtype_code(q_out.dtype), _stream()), "rope_cache")
+
+
 def gemm_simt(a: torch.Tensor, w: torch.Tensor, *, epilogue: int = EPI_STORE,
               bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
               resid: Optional[torch.Tensor] = None, activation: int = ACT_SILU) -> None:
@@ -436,7 +503,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_pool: 
               num_heads: int, num_kv_heads: int, head_dim: int, scale: float, window: int = 0,
               value_dim: Optional[int] = None, keep_first: int = 0, sink: bool = False, chunk: int = 0,
               out_scale: float = 1.0, sink_values: Optional[torch.Tensor] = None,
-              gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
+              gate: Optional[torch.Tensor] = None, gate_offset: int = 0, gate_per_head: bool = False) -> None:
     """Causal grouped-query attention of every token of the step over its request's pages.
     ``value_dim``: a value row's size (default d); ``keep_first``: with a window, that many
     first keys stay visible; ``sink``: one is added to the softmax's denominator; ``chunk``:
@@ -444,11 +511,11 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_pool: 
     (chunks counted from position 0); ``out_scale`` multiplies the output.  ``sink_values``
     float32 [heads]: exp(sink_h) joins head h's denominator instead of one.  ``gate`` float32
     [tokens, width]: the output is multiplied by the sigmoid of the heads * value_dim values that
-    start at column ``gate_offset`` of the token's row."""
+    start at column ``gate_offset`` of the token's row (``gate_per_head``: of heads values, one for a whole head)."""
     fn = _function("attention", "vipera_attention_gated",
                    [_c_void, _c_void, _c_int, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int,
                     _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void,
-                    _c_void, ctypes.c_longlong, _c_void])
+                    _c_void, ctypes.c_longlong, _c_int, _c_void])
     if chunk and window:
         raise InvalidArgumentError("attention: a mask is a window or chunks, not both")
     count = q.shape[0]
@@ -466,19 +533,15 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_pool: 
                                    "[pages, page_size, kv_heads, value size]")
     if sink_values is not None and sink_values.numel() != num_heads:
         raise InvalidArgumentError("attention: one sink score per query head")
-    gate_pointer, gate_stride = None, 0
-    if gate is not None:
-        if gate.dim() != 2 or gate.shape[0] != count or gate.stride(1) != 1 or \
-                not 0 <= gate_offset <= gate.shape[1] - num_heads * value_dim:
-            raise InvalidArgumentError("attention: the gate must hold heads * value size values per token")
-        gate_pointer = _gpu(gate, "gate", torch.float32) + 4 * int(gate_offset)
-        gate_stride = int(gate.stride(0))
+    gate_pointer, gate_stride = _gate_pointer(gate, gate_offset, count, num_heads * (1 if gate_per_head else value_dim),
+                                              "attention")
     _check(fn(_gpu(q, "q"), _gpu(out, "out"), dtype_code(q.dtype), _gpu(k_pool, "k_pool"), _gpu(v_pool, "v_pool"),
               _gpu(token_seq, "token_seq", torch.int32), _gpu(positions, "positions", torch.int32),
               _gpu(block_table, "block_table", torch.int32), block_table.shape[1], page_size, count,
               num_heads, num_kv_heads, head_dim, value_dim, float(scale), int(window or 0),
               int(keep_first or 0) if window else 0, 1 if sink else 0, int(chunk or 0), float(out_scale),
-              _opt(sink_values, "sink_values", torch.float32), gate_pointer, gate_stride, _stream()), "attention")
+              _opt(sink_values, "sink_values", torch.float32), gate_pointer, gate_stride, int(bool(gate_per_head)),
+              _stream()), "attention")
 
 
 # ----------------------------------------------------------------------------------------
@@ -772,13 +835,13 @@ def _gate_pointer(gate: Optional[torch.Tensor], gate_offset: int, rows: int, wid
     if gate is None:
         return None, 0
     if gate.dim() != 2 or gate.shape[0] != rows or gate.stride(1) != 1 or not 0 <= gate_offset <= gate.shape[1] - width:
-        raise InvalidArgumentError(f"{what}: the gate must hold heads * value size values per token")
+        raise InvalidArgumentError(f"{what}: the gate must hold a value per head, or per head and value, for every token")
     return _gpu(gate, "gate", torch.float32) + 4 * int(gate_offset), int(gate.stride(0))
 
 
-def attention_tc_takes_gate(gate: Optional[torch.Tensor], gate_offset: int) -> bool:
-    """The tensor-core ending reads the gate four values at a time."""
-    return gate is None or (gate_offset % 4 == 0 and gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0)
+def attention_tc_takes_gate(gate: Optional[torch.Tensor], gate_offset: int, gate_per_head: bool = False) -> bool:
+    """The tensor-core ending reads a gate of single values four at a time."""
+    return gate is None or gate_per_head or (gate_offset % 4 == 0 and gate.stride(0) % 4 == 0 and gate.data_ptr() % 16 == 0)
 
 
 def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, *,
@@ -786,7 +849,7 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, 
                       num_entries: int, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                       window: int = 0, skip_single: bool = False, keep_first: int = 0, sink: bool = False,
                       mask_chunk: int = 0, sink_values: Optional[torch.Tensor] = None,
-                      gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
+                      gate: Optional[torch.Tensor] = None, gate_offset: int = 0, gate_per_head: bool = False) -> None:
     """Flash-style attention of a step whose entries bring any number of tokens (bfloat16,
     head sizes 64 and 128), on tcgen05 with accumulators in tensor memory
     (VIPERA_ATTENTION_TC=0 keeps it on the mma.sync kernel).
@@ -796,8 +859,8 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, 
     a window: a query sees the earlier keys of its own chunk of that many positions; the kernels
     take it as a negative window).  ``sink_values`` float32 [heads] (a learned sink: exp(sink_h) joins
     head h's denominator) and ``gate`` (float32 [tokens, width]: the output is multiplied by the sigmoid
-    of the heads * d values from column ``gate_offset`` on) are served by the tcgen05 kernel's ending,
-    with a plain window only."""
+    of the heads * d values from column ``gate_offset`` on, or with ``gate_per_head`` of the heads values from
+    there on, one for a whole head) are served by the tcgen05 kernel's ending, with a plain window only."""
     if mask_chunk:
         if window:
             raise InvalidArgumentError("attention_prefill: a mask is a window or chunks, not both")
@@ -818,15 +881,18 @@ def attention_prefill(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, 
     skip = 1 if skip_single else 0
     keep_first = int(keep_first or 0) if window > 0 else 0
     if sink_values is not None or gate is not None:
-        if keep_first or window < 0 or (sink and sink_values is None) or not attention_tc_takes_gate(gate, gate_offset):
+        if keep_first or window < 0 or (sink and sink_values is None) or \
+                not attention_tc_takes_gate(gate, gate_offset, gate_per_head):
             raise UnsupportedError("attention_prefill: a learned sink and an output gate come with a plain window only")
         if sink_values is not None and sink_values.numel() != num_heads:
             raise InvalidArgumentError("attention_prefill: one sink score per query head")
-        gate_pointer, gate_stride = _gate_pointer(gate, gate_offset, count, num_heads * head_dim, "attention_prefill")
+        gate_pointer, gate_stride = _gate_pointer(gate, gate_offset, count, num_heads * (1 if gate_per_head else head_dim),
+                                                  "attention_prefill")
         fn = _function("attention_tc", "vipera_attention_prefill_tc_gated",
-                       kinds + [_c_int, _c_int, _c_void, _c_void, ctypes.c_longlong, _c_void, _c_void])
+                       kinds + [_c_int, _c_int, _c_void, _c_void, ctypes.c_longlong, _c_int, _c_void, _c_void])
         _check(fn(*pointers, *sizes, k_pool.shape[0], skip, _opt(sink_values, "sink_values", torch.float32), gate_pointer,
-                  gate_stride, kernel_status_word(q.device).data_ptr(), _stream()), "attention_prefill_tc")
+                  gate_stride, int(bool(gate_per_head)), kernel_status_word(q.device).data_ptr(), _stream()),
+               "attention_prefill_tc")
         return
     if keep_first or sink:
         fn = _function("attention_mma", "vipera_attention_prefill_kept", kinds + [_c_int, _c_int, _c_int, _c_void])
@@ -902,7 +968,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v
                      head_dim: int, scale: float, window: int, chunk: int, num_splits: int,
                      scratch: torch.Tensor, entry_starts: Optional[torch.Tensor] = None, keep_first: int = 0,
                      sink: bool = False, mask_chunk: int = 0, sink_values: Optional[torch.Tensor] = None,
-                     gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
+                     gate: Optional[torch.Tensor] = None, gate_offset: int = 0, gate_per_head: bool = False) -> None:
     """Split-key attention of the entries that bring one token (bfloat16, head sizes 64 and
     128); the partial results of the splits are combined by a second kernel.  Without
     ``entry_starts`` every entry brings one token (q and out are [entries, heads * d], positions
@@ -913,7 +979,8 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v
     the scratch is sized for ``num_splits + 1``) and ``sink`` (one added to the softmax's denominator).
     ``mask_chunk``: instead of a window, chunks of that many positions (passed on as a negative window).
     ``sink_values`` float32 [heads]: a learned sink per query head; ``gate`` float32 [rows of q, width]: the
-    output is multiplied by the sigmoid of the heads * d values from column ``gate_offset`` on."""
+    output is multiplied by the sigmoid of the heads * d values from column ``gate_offset`` on (``gate_per_head``:
+    of the heads values from there on, one for a whole head)."""
     if mask_chunk:
         if window:
             raise InvalidArgumentError("attention_decode: a mask is a window or chunks, not both")
@@ -921,10 +988,11 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v
     fn = _function("attention_mma", "vipera_attention_decode_gated",
                    [_c_void, _c_void, _c_void, _c_void, _c_void, _c_void, _c_int, _c_int, _c_int, _c_int, _c_int,
                     _c_int, _c_float, _c_int, _c_int, _c_int, _c_void, ctypes.c_size_t, _c_void, _c_int, _c_int,
-                    _c_void, _c_void, ctypes.c_longlong, _c_void])
+                    _c_void, _c_void, ctypes.c_longlong, _c_int, _c_void])
     if sink_values is not None and sink_values.numel() != num_heads:
         raise InvalidArgumentError("attention_decode: one sink score per query head")
-    gate_pointer, gate_stride = _gate_pointer(gate, gate_offset, q.shape[0], num_heads * head_dim, "attention_decode")
+    gate_pointer, gate_stride = _gate_pointer(gate, gate_offset, q.shape[0], num_heads * (1 if gate_per_head else head_dim),
+                                              "attention_decode")
     if head_dim not in MMA_HEAD_DIMS:
         raise UnsupportedError(f"attention_decode: head size {head_dim} (built: 64, 128)")
     count = block_table.shape[0]
@@ -942,7 +1010,7 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_pool: torch.Tensor, v
               num_heads, num_kv_heads, head_dim, float(scale), int(window or 0), int(chunk), int(num_splits),
               _gpu(scratch, "scratch", torch.float32), scratch.numel(), _opt(entry_starts, "entry_starts", torch.int32),
               int(keep_first or 0) if window > 0 else 0, 1 if sink else 0, _opt(sink_values, "sink_values", torch.float32),
-              gate_pointer, gate_stride, _stream()), "attention_decode", kernels=2)
+              gate_pointer, gate_stride, int(bool(gate_per_head)), _stream()), "attention_decode", kernels=2)
 
 
 def attention_decode_scratch_floats(num_entries: int, num_heads: int, head_dim: int, num_splits: int) -> int:
@@ -1560,6 +1628,97 @@ def gated_norm_add(branch: torch.Tensor, parts: int, gate: Optional[torch.Tensor
 
 
 # ----------------------------------------------------------------------------------------
+# Mamba-2's recurrence
+# ----------------------------------------------------------------------------------------
+class _Mamba2Params(ctypes.Structure):
+    _fields_ = [
+        ("xbc", _c_void), ("xbc_width", ctypes.c_longlong), ("proj", _c_void), ("proj_width", ctypes.c_longlong),
+        ("z_off", _c_int), ("dt_off", _c_int), ("dt_bias", _c_void), ("a", _c_void), ("d", _c_void), ("state", _c_void),
+        ("entry_starts", _c_void), ("state_slots", _c_void), ("fresh", _c_void), ("y", _c_void), ("norm_weight", _c_void),
+        ("out", _c_void), ("chunk_state", _c_void), ("chunk_decay", _c_void),
+        ("heads", _c_int), ("vdim", _c_int), ("groups", _c_int), ("states", _c_int), ("norm_groups", _c_int),
+        ("num_entries", _c_int), ("num_tokens", _c_int), ("num_jobs", _c_int), ("heads_per_block", _c_int),
+        ("single_only", _c_int), ("eps", _c_float),
+    ]
+
+
+MAMBA2_CHUNK, MAMBA2_MAX_STATE = 128, 256   # kChunk, kMaxState in mamba2.cu
+MAMBA2_COLS = 64                            # kCols: value columns of a block
+
+
+def mamba2_jobs(tokens: int, num_entries: int) -> int:
+    """The most chunks a step of `tokens` tokens in `num_entries` entries has."""
+    return tokens // MAMBA2_CHUNK + num_entries
+
+
+@functools.lru_cache(maxsize=4096)
+def mamba2_heads_per_block(jobs: int, heads: int, groups: int, vdim: int, sm_count: int) -> int:
+    """How many heads of a group a block of the chunked form works on: more share the scores, as long as
+    the blocks still fill the GPU twice."""
+    tiles = -(-vdim // MAMBA2_COLS)
+    for wanted in (8, 4, 2):
+        if (heads // groups) % wanted == 0 and jobs * (heads // wanted) * tiles >= 2 * sm_count:
+            return wanted
+    return 1
+
+
+def mamba2(xbc: torch.Tensor, proj: torch.Tensor, *, z_off: int, dt_off: int, heads: int, vdim: int, groups: int,
+           states: int, dt_bias: torch.Tensor, a: torch.Tensor, d: torch.Tensor, state: torch.Tensor,
+           entry_starts: torch.Tensor, state_slots: torch.Tensor, fresh: torch.Tensor, num_entries: int,
+           any_single: bool, y: torch.Tensor, norm_weight: torch.Tensor, norm_groups: int, eps: float,
+           out: torch.Tensor, chunks=None) -> None:
+    """Mamba-2's recurrence over a step, its gate and its norm.  ``xbc`` [tokens, heads * vdim + 2 groups *
+    states] (x, B, C past convolution and activation, in the run's type); ``proj`` float32 [tokens, width] with
+    the gate z at column ``z_off`` and the raw step sizes at ``dt_off``; ``state`` float32 [slots, heads *
+    states * vdim], read where an entry is not fresh and left as the entry's last token leaves it.  ``y``
+    float32 [tokens, heads * vdim] is scratch; ``out`` (xbc's type) receives ``y * silu(z)`` divided by its root
+    mean square in ``norm_groups`` parts, times ``norm_weight``.  ``chunks`` (bfloat16: float32 tensors [jobs,
+    heads * states * vdim] and [jobs, heads], jobs >= mamba2_jobs(...)): entries of several tokens run as chunks
+    side by side; ``any_single`` then says whether there are entries of one token beside them."""
+    fn = _function("mamba2", "vipera_mamba2", [ctypes.POINTER(_Mamba2Params), _c_int, _c_int, _c_void])
+    _check_struct("mamba2", "vipera_mamba2_params_size", _Mamba2Params)
+    tokens, inner = xbc.shape[0], heads * vdim
+    if states > MAMBA2_MAX_STATE:
+        raise UnsupportedError(f"mamba2: a state of {states} rows; the kernels take up to {MAMBA2_MAX_STATE}")
+    if heads % groups or inner % norm_groups or xbc.shape[1] != inner + 2 * groups * states:
+        raise InvalidArgumentError("mamba2: xbc must be [tokens, heads * vdim + 2 groups * states]")
+    if proj.dim() != 2 or proj.shape[0] != tokens or not 0 <= z_off <= proj.shape[1] - inner or \
+            not 0 <= dt_off <= proj.shape[1] - heads:
+        raise InvalidArgumentError("mamba2: proj must hold the gate and the step sizes of every token")
+    if tuple(y.shape) != (tokens, inner) or tuple(out.shape) != (tokens, inner) or out.dtype != xbc.dtype:
+        raise InvalidArgumentError("mamba2: y and out must be [tokens, heads * vdim]")
+    if state.dim() != 2 or state.shape[1] != heads * states * vdim or norm_weight.numel() != inner or \
+            any(v.numel() != heads for v in (dt_bias, a, d)):
+        raise InvalidArgumentError("mamba2: state rows, norm weight or the numbers per head have the wrong size")
+    if entry_starts.numel() < num_entries + 1 or state_slots.numel() < num_entries or fresh.numel() < num_entries:
+        raise InvalidArgumentError("mamba2: the step's description is too short for its entries")
+    p = _Mamba2Params()
+    p.xbc, p.xbc_width = _gpu(xbc, "xbc"), int(xbc.shape[1])
+    p.proj, p.proj_width = _gpu(proj, "proj", torch.float32), int(proj.shape[1])
+    p.z_off, p.dt_off = int(z_off), int(dt_off)
+    p.dt_bias, p.a, p.d = _gpu(dt_bias, "dt_bias", torch.float32), _gpu(a, "a", torch.float32), _gpu(d, "d", torch.float32)
+    p.state = _gpu(state, "state", torch.float32)
+    p.entry_starts = _gpu(entry_starts, "entry_starts", torch.int32)
+    p.state_slots = _gpu(state_slots, "state_slots", torch.int32)
+    p.fresh = _gpu(fresh, "fresh", torch.int32)
+    p.y, p.out = _gpu(y, "y", torch.float32), _gpu(out, "out")
+    p.norm_weight, p.norm_groups, p.eps = _gpu(norm_weight, "norm_weight", torch.float32), int(norm_groups), float(eps)
+    p.heads, p.vdim, p.groups, p.states = int(heads), int(vdim), int(groups), int(states)
+    p.num_entries, p.num_tokens = int(num_entries), int(tokens)
+    launched = 2
+    if chunks is not None:
+        sums, decays = chunks
+        jobs = mamba2_jobs(tokens, num_entries)
+        if xbc.dtype != torch.bfloat16 or sums.numel() < jobs * heads * states * vdim or decays.numel() < jobs * heads:
+            raise InvalidArgumentError("mamba2: the chunked form runs in bfloat16 and needs room for every chunk of the step")
+        p.chunk_state, p.chunk_decay = _gpu(sums, "chunk states", torch.float32), _gpu(decays, "chunk decays", torch.float32)
+        p.num_jobs = jobs
+        p.heads_per_block = mamba2_heads_per_block(jobs, int(heads), int(groups), int(vdim), sm_count(xbc.device))
+        launched = 4 + int(bool(any_single))
+    _check(fn(ctypes.byref(p), dtype_code(xbc.dtype), int(bool(any_single)), _stream()), "mamba2", kernels=launched)
+
+
+# ----------------------------------------------------------------------------------------
 # attention over a cached low-rank latent
 # ----------------------------------------------------------------------------------------
 class _LatentParams(ctypes.Structure):
@@ -1810,7 +1969,7 @@ class _MoeParams(ctypes.Structure):
         ("gate_group", _c_int), ("tile_rows", _c_int), ("padded", _c_int),
         ("correction", _c_void), ("identity", _c_int), ("always", _c_int), ("slots", _c_int), ("gated", _c_int),
         ("route_scale", _c_float), ("renorm_eps", _c_float),
-        ("always_gate", _c_int), ("unit_limit", _c_void), ("unit_slope", _c_float),
+        ("always_gate", _c_int), ("unit_limit", _c_void), ("unit_slope", _c_float), ("input_weight", _c_int),
     ]
 
 
@@ -1876,7 +2035,7 @@ def moe(h: torch.Tensor, *, router: torch.Tensor, gate_up: torch.Tensor, down: t
         xs: Optional[torch.Tensor] = None, ys: Optional[torch.Tensor] = None, gated: bool = True,
         correction: Optional[torch.Tensor] = None, identity: int = 0, always: int = 0, route_scale: float = 1.0,
         renorm_eps: float = 0.0, logit_scores: bool = False, always_gate: bool = False,
-        unit_limit: Optional[torch.Tensor] = None, unit_slope: float = 0.0) -> None:
+        unit_limit: Optional[torch.Tensor] = None, unit_slope: float = 0.0, input_weight: bool = False) -> None:
     """A mixture of gated units over a step.  ``h`` [tokens, hidden]; ``router`` float32 [experts,
     hidden]; ``gate_up`` [experts, 2 ff, hidden] (``gate_group`` gate rows, then the up rows of the
     same features, and so on) and ``down`` [experts, hidden, ff] in h's type.  ``chosen`` int32 and
@@ -1896,7 +2055,8 @@ def moe(h: torch.Tensor, *, router: torch.Tensor, gate_up: torch.Tensor, down: t
     ``route_scale`` multiplies them.  ``logit_scores``: the scores are the logits themselves, and the
     weights the softmax over the chosen ones.  ``always_gate``: ``router`` has one row more, and the
     always-used units' weight is the sigmoid of its product with h.  Activation ACT_CLAMPED: gated units
-    with the bounds ``unit_limit`` (float32, one per unit with matrices) and ``unit_slope``."""
+    with the bounds ``unit_limit`` (float32, one per unit with matrices) and ``unit_slope``.
+    ``input_weight``: a chosen expert's weight multiplies what it reads and not its output."""
     fn = _function("moe", "vipera_moe", [ctypes.POINTER(_MoeParams), _c_int, _c_void])
     _check_struct("moe", "vipera_moe_params_size", _MoeParams)
     tokens, hidden = h.shape
@@ -1941,7 +2101,7 @@ def moe(h: torch.Tensor, *, router: torch.Tensor, gate_up: torch.Tensor, down: t
     p.groups, p.keep, p.group_top, p.max_tiles = int(groups), int(keep), int(group_top), int(tiles)
     p.scores = 2 if logit_scores else int(bool(softmax_scores))
     p.renormalize, p.activation = int(bool(renormalize)), int(activation)
-    p.always_gate, p.unit_slope = int(bool(always_gate)), float(unit_slope)
+    p.always_gate, p.unit_slope, p.input_weight = int(bool(always_gate)), float(unit_slope), int(bool(input_weight))
     p.unit_limit = _opt(unit_limit, "unit_limit", torch.float32)
     p.gate_group, p.tile_rows, p.padded = int(gate_group), int(tile_rows), int(padded)
     if not padded:

@@ -22,6 +22,7 @@ from ..kernels import ops
 from ..weights import TensorSpec
 from .base import Mixer, PagedKV
 from .linear import Linear, NormedInput
+from .rotary import QueryFactor
 
 
 class GQAttention(Mixer):
@@ -43,14 +44,21 @@ class GQAttention(Mixer):
     ``sink = "learned"`` (the sink's score is a number per query head, ``<prefix>.sink.weight`` [heads]:
     ``exp(sink_h)`` joins the denominator, unscaled); ``output_gate`` (the concatenated heads are
     multiplied by ``sigmoid(W_g h)``, ``<prefix>.<gate_name>.weight`` [heads * value_dim, hidden],
-    ``gate_name`` ``g`` by default; the gate's rows join the q/k/v product); ``value_mix``:
+    ``gate_name`` ``g`` by default; the gate's rows join the q/k/v product; ``output_gate = "heads"``: one number
+    per head, the matrix being [heads, hidden]); ``head_norm`` with ``norm_eps`` (each query and key head is
+    divided by its own root mean square and multiplied by a weight per value that all heads share,
+    ``<q>.norm.weight`` and ``<k>.norm.weight`` [head_dim], before the rotation); ``query_temperature``
+    (``{"coef", "every"}``, with ``max_positions``: the query at position p is multiplied by
+    ``1 + coef ln(floor((p + 1) / every) + 1)``); ``value_mix``:
     ``"source"`` publishes the values of the step's tokens as projected, ``"blend"`` caches
     ``(1 - b) v + b v_source`` with ``b = <prefix>.vmix.weight`` (a single number) and ``v_source`` what
     the source layer published for the same token earlier in the step (both kinds hold the tensor;
-    the source does not read it)."""
+    the source does not read it).  Handed no stream, the mixer leaves its output as rows (``rows_name``: the
+    buffer they are in)."""
 
     kernels = ("rope_cache", "attention", "attention_mma", "attention_tc")
     takes_lazy_input = True
+    leaves_rows = True   # forward(ctx, h, None, ...) returns (rows [tokens, hidden] float32, 1)
     # With mixed head weights: steps of this many tokens and more that bring portions run every
     # (query head, KV head) pair through the tensor-core flash kernel; shorter ones and steps of
     # single tokens run the split-key kernels.
@@ -78,12 +86,16 @@ class GQAttention(Mixer):
         if params.get("row_norm", False):
             schema[f"{prefix}.{qn}.norm.weight"] = TensorSpec((q_width,), init="norm")
             schema[f"{prefix}.{kn}.norm.weight"] = TensorSpec((kv_width,), init="norm")
+        if params.get("head_norm", False):
+            schema[f"{prefix}.{qn}.norm.weight"] = TensorSpec((d,), init="norm", store="float32")
+            schema[f"{prefix}.{kn}.norm.weight"] = TensorSpec((d,), init="norm", store="float32")
         if params.get("talking_heads", False):
             schema[f"{prefix}.talk.weight"] = TensorSpec((params["num_heads"], params["num_heads"]), init="mix")
         if params.get("sink") == "learned":
             schema[f"{prefix}.sink.weight"] = TensorSpec((params["num_heads"],), init="sink", store="float32")
         if params.get("output_gate", False):
-            schema[f"{prefix}.{params.get('gate_name', 'g')}.weight"] = TensorSpec((params["num_heads"] * dv, hidden))
+            gate_rows = params["num_heads"] * (1 if params["output_gate"] == "heads" else dv)
+            schema[f"{prefix}.{params.get('gate_name', 'g')}.weight"] = TensorSpec((gate_rows, hidden))
         if params.get("value_mix"):
             schema[f"{prefix}.vmix.weight"] = TensorSpec((), init="blend", store="float32")
         if params.get("qkv_bias", False):
@@ -108,6 +120,14 @@ class GQAttention(Mixer):
         elif params.get("sink") not in (None, False, True):
             raise UnsupportedError(f"{prefix}: sink is true or \"learned\", not {params.get('sink')!r}")
         self.gated = bool(params.get("output_gate", False))
+        if params.get("output_gate", False) not in (None, False, True, "heads"):
+            raise UnsupportedError(f"{prefix}: output_gate is true or \"heads\", not {params['output_gate']!r}")
+        self.gate_per_head = params.get("output_gate", False) == "heads"
+        self.rows_name = str(params.get("rows_name", "attention.rows"))
+        self.head_norm = bool(params.get("head_norm", False))
+        self.q_factor = None
+        if params.get("query_temperature"):
+            self.q_factor = QueryFactor(params["query_temperature"], int(params["max_positions"]), device)
         self.value_mix = params.get("value_mix") or None
         if self.value_mix not in (None, "source", "blend"):
             raise UnsupportedError(f"{prefix}: value_mix is \"source\" or \"blend\", not {self.value_mix!r}")
@@ -139,6 +159,18 @@ class GQAttention(Mixer):
         if self.row_norm:
             self.q_norm = tensors[f"{prefix}.{qn}.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
             self.k_norm = tensors[f"{prefix}.{kn}.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
+        if self.head_norm:
+            if self.row_norm or self.values_from_keys or self.value_mix:
+                raise UnsupportedError("attention: a norm per head does not come with a norm over whole rows, blended values "
+                                       "or values that are the keys")
+            self.q_norm = tensors[f"{prefix}.{qn}.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
+            self.k_norm = tensors[f"{prefix}.{kn}.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
+        if self.q_factor is not None and (self.row_norm or self.values_from_keys or self.value_mix):
+            raise UnsupportedError("attention: queries that grow with their position do not come with a norm over whole rows, "
+                                   "blended values or values that are the keys")
+        if self.gated and self.sink and self.sink_values is None:
+            # the gated kernels know a score per head: a sink of score 0 is a learned one that is 0 everywhere
+            self.sink_values = torch.zeros(self.num_heads, dtype=torch.float32, device=device)
         if (self.gated or self.value_mix) and (self.values_from_keys or self.row_norm):
             raise UnsupportedError("attention: an output gate or blended values do not come with a norm over whole "
                                    "rows or values that are the keys")
@@ -164,7 +196,7 @@ class GQAttention(Mixer):
                             and not self.keep_first and not self.sink and self.head_dim % 16 == 0
                             and not self.chunk and not self.values_from_keys and not self.row_norm
                             and self.talk is None and self.out_scale == 1.0 and not self.gated
-                            and self.value_mix is None)
+                            and self.value_mix is None and not self.head_norm and self.q_factor is None)
 
     def kernel_families(self):
         # the tensor-core attention kernels serve bfloat16 with head sizes 64 and 128; everything
@@ -187,6 +219,8 @@ class GQAttention(Mixer):
         prepare = getattr(self.position, "prepare", None)
         if prepare is not None:
             prepare(max_positions)
+        if self.q_factor is not None:
+            self.q_factor.prepare(max_positions)
 
     @classmethod
     def cache_request_for(cls, params):
@@ -202,11 +236,21 @@ class GQAttention(Mixer):
         q_width = params["num_heads"] * params["head_dim"]
         qkv_width = q_width + params["num_kv_heads"] * (params["head_dim"] + dv)
         if params.get("output_gate", False):
-            qkv_width += params["num_heads"] * dv
+            qkv_width += params["num_heads"] * (1 if params["output_gate"] == "heads" else dv)
         if params.get("value_mix"):
             qkv_width += params["num_kv_heads"] * dv   # the published values, 32-bit
         # q and the attention's output in the run's type, and the 32-bit q/k/v product of the unfused route
-        return tokens * ((q_width + params["num_heads"] * dv) * element_bytes + qkv_width * 4)
+        # (and the rows it leaves where an arrangement takes rows)
+        return tokens * ((q_width + params["num_heads"] * dv) * element_bytes + qkv_width * 4 + params["hidden_size"] * 4)
+
+    def _output(self, ctx, mixed, residual):
+        """The output product: added into the stream, or left as rows where there is none."""
+        if residual is None:
+            rows = ctx.workspace.get(self.rows_name, (ctx.num_tokens, self.hidden), torch.float32)
+            self.out(ctx, mixed, epilogue=ops.EPI_STORE, out=rows)
+            return rows, 1
+        self.out(ctx, mixed, epilogue=ops.EPI_RESIDUAL, resid=residual)
+        return None
 
     def forward(self, ctx, h, residual, cache, writes_cache):
         count = ctx.num_tokens
@@ -229,8 +273,7 @@ class GQAttention(Mixer):
                                epilogue=ops.GEMV_ROPE_CACHE, bias=self.qkv.bias, rope=rope)
             mixed = ws.get("attention.out", (count, heads * d), ctx.dtype)
             self._attend(ctx, q, mixed, cache, table)
-            self.out(ctx, mixed, epilogue=ops.EPI_RESIDUAL, resid=residual)
-            return
+            return self._output(ctx, mixed, residual)
         if (self.common_form and ctx.dtype == torch.bfloat16 and style in (ops.ROPE_NONE, ops.ROPE_NEOX)
                 and self.qkv.tensor_core
                 and ops.gemm_tc_rope_takes(count, self.qkv.out_features, self.qkv.in_features, d)):
@@ -243,8 +286,7 @@ class GQAttention(Mixer):
                              page_size=cache.page_size, write_cache=writes_cache)
             mixed = ws.get("attention.out", (count, heads * d), ctx.dtype)
             self._attend(ctx, q, mixed, cache, table)
-            self.out(ctx, mixed, epilogue=ops.EPI_RESIDUAL, resid=residual)
-            return
+            return self._output(ctx, mixed, residual)
         qkv = ws.get("attention.qkv", (count, self.qkv.out_features), torch.float32)
         self.qkv(ctx, h, epilogue=ops.EPI_STORE, out=qkv)
         if self.row_norm or self.values_from_keys:
@@ -258,8 +300,7 @@ class GQAttention(Mixer):
                            block_table=table, page_size=cache.page_size, write_cache=writes_cache)
             mixed = ws.get("attention.out", (count, heads * dv), ctx.dtype)
             self._attend(ctx, q, mixed, cache, table)
-            self.out(ctx, mixed, epilogue=ops.EPI_RESIDUAL, resid=residual)
-            return
+            return self._output(ctx, mixed, residual)
         if style is None:
             # An encoding the fused kernel does not know: the part applies it to the 32-bit
             # product itself, then the kernel only converts and stores.
@@ -269,7 +310,13 @@ class GQAttention(Mixer):
             style, cos, sin = ops.ROPE_NONE, None, None
         else:
             cos, sin = self.position.tables()
-        if self.gated or self.value_mix:
+        if self.head_norm or self.q_factor is not None:
+            ops.head_rows(qkv, q, num_heads=heads, num_kv_heads=kv_heads, head_dim=d, value_dim=dv,
+                          rot_dims=self.rot_dims if style != ops.ROPE_NONE else 0, positions=ctx.positions, cos=cos, sin=sin,
+                          style=style, k_pool=cache.k, v_pool=cache.v, token_entry=ctx.token_entry, block_table=table,
+                          page_size=cache.page_size, write_cache=writes_cache, q_norm=self.q_norm, k_norm=self.k_norm,
+                          eps=self.norm_eps, q_factor=None if self.q_factor is None else self.q_factor.table())
+        elif self.gated or self.value_mix:
             publish = blend_with = None
             if self.value_mix == "source":
                 publish = ws.get("attention.value_mix", (count, kv_heads * dv), torch.float32)
@@ -291,7 +338,7 @@ class GQAttention(Mixer):
                            page_size=cache.page_size, write_cache=writes_cache, value_dim=dv, rot_dims=self.rot_dims)
         mixed = ws.get("attention.out", (count, heads * dv), ctx.dtype)
         self._attend(ctx, q, mixed, cache, table, gate=qkv if self.gated else None)
-        self.out(ctx, mixed, epilogue=ops.EPI_RESIDUAL, resid=residual)
+        return self._output(ctx, mixed, residual)
 
     def _attend(self, ctx, q, mixed, cache, table, gate=None):
         """Choose the attention kernel: on the bfloat16 path with a head size the tensor-core
@@ -338,7 +385,7 @@ class GQAttention(Mixer):
         # a learned sink and an output gate are endings of the tcgen05 flash kernel and of the split-key
         # kernel's combine (plain windows only); elsewhere they run through the general kernel
         extended = self.sink_values is not None or gate is not None
-        extended_ok = (not self.keep_first and not self.chunk and ops.attention_tc_takes_gate(gate, self.gate_offset)
+        extended_ok = (not self.keep_first and not self.chunk and ops.attention_tc_takes_gate(gate, self.gate_offset, self.gate_per_head)
                        and d in ops.TC_ATTENTION_HEAD_DIMS and os.environ.get("VIPERA_ATTENTION_TC", "1") != "0")
         if (self.out_scale == 1.0 and ctx.dtype == torch.bfloat16 and d in ops.MMA_HEAD_DIMS and self.value_dim == d
                 and (not extended or extended_ok)):
@@ -346,7 +393,7 @@ class GQAttention(Mixer):
             # the kept keys as tiles of their own, the split-key kernel as a split of its own); the
             # tcgen05 flash kernel serves attention without them.
             kept = dict(keep_first=self.keep_first, sink=self.sink, mask_chunk=self.chunk, sink_values=self.sink_values,
-                        gate=gate, gate_offset=self.gate_offset)
+                        gate=gate, gate_offset=self.gate_offset, gate_per_head=self.gate_per_head)
             places = 1 if self.keep_first else 0
             if ctx.all_single:
                 chunk, splits = ops.decode_splits(ctx.num_entries, kv_heads, max(ctx.max_kv_len, 1),
@@ -380,7 +427,7 @@ class GQAttention(Mixer):
                       block_table=table, num_heads=heads, num_kv_heads=kv_heads, head_dim=d,
                       scale=self.scale, window=window, value_dim=self.value_dim, keep_first=self.keep_first,
                       sink=self.sink, chunk=self.chunk, out_scale=self.out_scale, sink_values=self.sink_values,
-                      gate=gate, gate_offset=self.gate_offset)
+                      gate=gate, gate_offset=self.gate_offset, gate_per_head=self.gate_per_head)
 
 
 MIXERS.register("gqa_attention", GQAttention)

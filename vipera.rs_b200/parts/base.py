@@ -15,7 +15,9 @@ Mixer           ``cache_request()`` says what the mixer keeps between steps (pag
 FeedForward     ``forward(ctx, h, residual)`` adds its output into ``residual`` in place.
                 (A mixer or feed-forward that sets ``leaves_rows`` may be handed None as its
                 ``residual``: it then leaves its output and returns (rows [tokens, parts * hidden]
-                float32, parts), the output being the sum of a token's parts in their order.)
+                float32, parts), the output being the sum of a token's parts in their order.  One that
+                sets ``leaves_branches`` returns a list of branches instead: (rows, parts, scale per
+                channel or None, eps or None), with an eps each divided by its own root mean square.)
 Block           ``forward(ctx, residual, cache, writes_cache)`` arranges the four.
 
 The reference's seam between runtime and backend is the same in spirit: the backend turns

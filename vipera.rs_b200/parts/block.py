@@ -326,12 +326,22 @@ class SandwichBlock(Block):
 
 class PendingJoin:
     """Branches of a layer that have been computed and not yet added to the stream: ``(rows, parts,
-    scale)`` each, ``x += scale * sum of the parts``.  Whoever reads the stream next adds them on the way:
+    scale)`` each, ``x += scale * sum of the parts``, or ``(rows, parts, scale, eps)`` where the sum is
+    first divided by its root mean square.  Whoever reads the stream next adds them on the way:
     a ``parallel`` layer and the model's last norm in the kernel that computes their norms, anything else
     after ``settle``."""
 
     def __init__(self, branches):
         self.branches = list(branches)
+
+    @staticmethod
+    def add(ctx, residual, branch) -> None:
+        """One more branch for the stream, beside what is pending already."""
+        if ctx.pending is not None and len(ctx.pending.branches) >= 4:
+            PendingJoin.settle(ctx, residual)
+        if ctx.pending is None:
+            ctx.pending = PendingJoin([])
+        ctx.pending.branches.append(branch)
 
     @staticmethod
     def settle(ctx, residual) -> None:
@@ -370,9 +380,11 @@ class ParallelBlock(Block):
 
     (the second term only where the layer has a feed-forward).  ``params``: ``hidden_size`` and
     ``layer_scale`` (true: tensors ``<layer>.<mixer_scale>.weight`` and ``<layer>.<ffn_scale>.weight``
-    [hidden], the s above; false: 1).  The branches are left for the next reader of the stream to add
-    (``PendingJoin``): one kernel adds a layer's branches, with their scales and the sum over a token's
-    expert rows, and computes both norms of the next layer."""
+    [hidden], the s above; false: 1) and ``shared_norm`` (true: there is one norm, ``mixer_norm``, and both
+    sublayers read its output, ``x += s1 * mixer(N(x)) + s2 * ff(N(x))``).  The branches are left for the next
+    reader of the stream to add (``PendingJoin``): one kernel adds a layer's branches, with their scales and the
+    sum over a token's expert rows, and computes the next layer's norm or norms.  A mixer may leave branches of
+    its own (``leaves_branches``)."""
 
     roles = {"mixer_norm": NORMS, "mixer": MIXERS}
     optional_roles = {"ffn_norm": NORMS, "ffn": FEED_FORWARDS}
@@ -386,6 +398,8 @@ class ParallelBlock(Block):
         self.scales = {side: None for side in self.sides}
         if layer_spec.params.get("layer_scale", False):
             for side in self.sides:
+                if getattr(self._parts[side], "leaves_branches", False):
+                    raise UnsupportedError(f"{layer_spec.prefix}: a scale per channel on a mixer that leaves normed branches")
                 scale = tensors[f"{layer_spec.part_prefix(side + '_scale')}.weight"]
                 self.scales[side] = scale.to(device=device, dtype=torch.float32).contiguous()
 
@@ -398,6 +412,8 @@ class ParallelBlock(Block):
         roles = dict(cls.roles)
         if "ffn" in layer_spec.parts:
             roles.update(cls.optional_roles)
+            if layer_spec.params.get("shared_norm", False):
+                del roles["ffn_norm"]
         return roles
 
     @classmethod
@@ -422,22 +438,25 @@ class ParallelBlock(Block):
         return total
 
     def _branch(self, ctx, side, run):
-        """What one side adds to the stream.  A part that cannot leave rows adds into a cleared buffer."""
+        """What one side adds to the stream, a list of branches.  A part that cannot leave rows adds into a
+        cleared buffer."""
         part = self._parts[side]
+        if getattr(part, "leaves_branches", False):
+            return run(part, None)
         if getattr(part, "leaves_rows", False):
             rows, parts = run(part, None)
         else:
             rows, parts = ctx.workspace.get(f"block.{side}_rows", (ctx.num_tokens, self.hidden), torch.float32), 1
             rows.zero_()
             run(part, rows)
-        return rows, parts, self.scales[side]
+        return [(rows, parts, self.scales[side])]
 
     def forward(self, ctx, residual, cache, writes_cache):
-        norms = [self._parts[f"{side}_norm"] for side in self.sides]
+        norms = [self._parts[f"{side}_norm"] for side in self.sides if f"{side}_norm" in self._parts]
         inputs = PendingJoin.normed(ctx, residual, norms, ["block.h", "block.h2"][:len(norms)])
-        branches = [self._branch(ctx, "mixer", lambda part, into: part.forward(ctx, inputs[0], into, cache, writes_cache))]
+        branches = self._branch(ctx, "mixer", lambda part, into: part.forward(ctx, inputs[0], into, cache, writes_cache))
         if "ffn" in self._parts:
-            branches.append(self._branch(ctx, "ffn", lambda part, into: part.forward(ctx, inputs[1], into)))
+            branches = branches + self._branch(ctx, "ffn", lambda part, into: part.forward(ctx, inputs[-1], into))
         ctx.pending = PendingJoin(branches)
 
 

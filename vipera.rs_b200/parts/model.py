@@ -77,6 +77,10 @@ class DecoderModel:
             if entry.writes_cache:
                 self.cache_requests[entry.cache] = self.blocks[entry.layer].cache_request()
 
+    @property
+    def adds_embedding(self) -> bool:
+        return any(entry.adds_embedding for entry in self.spec.schedule)
+
     def prepare(self, max_positions: int) -> None:
         """Tell every part that sizes something by position (tables of a position encoding)
         how far the engine goes: positions below `max_positions`."""
@@ -126,12 +130,20 @@ class DecoderModel:
         [wanted rows, vocab], or None when no row is wanted."""
         ws = ctx.workspace
         residual = ws.get("model.residual", (ctx.num_tokens, self.spec.hidden_size), torch.float32)
-        ops.embed(self.embedding, ctx.tokens, residual, self.spec.embedding_scale)
+        embedded = None   # the stream before the first layer, kept where an entry adds it again
+        if self.adds_embedding:
+            embedded = ws.get("model.embedded", (ctx.num_tokens, self.spec.hidden_size), torch.float32)
+        ops.embed(self.embedding, ctx.tokens, residual, self.spec.embedding_scale,
+                  also=embedded if self.embedding_norm is None else None)
         if self.embedding_norm is not None:
             # in place: the normed rows are the stream the first layer reads, in 32-bit
             self.embedding_norm.forward(ctx, residual, residual)
+            if embedded is not None:
+                embedded.copy_(residual)
         ctx.pending = None
         for entry in self.spec.schedule:
+            if entry.adds_embedding:
+                PendingJoin.add(ctx, residual, (embedded, 1, None))
             if not self.blocks[entry.layer].takes_pending:
                 PendingJoin.settle(ctx, residual)
             self.blocks[entry.layer].forward(ctx, residual, caches.get(entry.cache), entry.writes_cache)

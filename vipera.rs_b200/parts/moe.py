@@ -27,7 +27,9 @@ further units with weight 1 (or, with ``shared_gate``, the sigmoid of one more r
 h), through the same tiles and products.  ``score`` = ``logit``: the choice is by the logits, the weights
 are the softmax over the chosen logits.  ``activation`` = ``clamped``: with g = G h bounded above by the
 unit's limit and u = U h held within it on both sides, ``D (g sigmoid(slope g) (u + 1))``; the shared
-unit has a limit of its own, and a feature filled up with zeros gives 0.
+unit has a limit of its own, and a feature filled up with zeros gives 0.  ``weight_on`` = ``input``: an
+expert's weight multiplies what it reads, ``D_e (act(w_e G_e h) * (w_e U_e h))``, in the ending of the first
+product (or, for the grouped products, as the tokens' rows are gathered).
 """
 from __future__ import annotations
 
@@ -50,6 +52,7 @@ class MixtureOfExperts(FeedForward):
     (default gate, up, down), ``gated`` (default true; false: no gate matrices), ``identity`` (default 0:
     the last that many of the ``experts`` router outputs have no matrices), ``correction`` (true: tensor
     ``<prefix>.correction.weight`` [experts]), ``route_scale`` (default 1), ``renorm_eps`` (default 0),
+    ``weight_on`` (``output``, the default, or ``input``),
     ``shared_size`` (default none: the inner size of a shared unit, tensors ``<prefix>.shared.<name>.weight``).
     Tensors: ``<prefix>.router.weight`` [experts, hidden] and, per expert k that has matrices,
     ``<prefix>.e<k>.<gate|up>.weight`` [intermediate, hidden] and ``<prefix>.e<k>.<down>.weight``
@@ -121,6 +124,9 @@ class MixtureOfExperts(FeedForward):
         self.activation = known[name]
         self.identity = int(params.get("identity") or 0)
         self.route_scale = float(params.get("route_scale", 1.0))
+        if params.get("weight_on", "output") not in ("output", "input"):
+            raise UnsupportedError(f"{prefix}: an expert's weight is on its output or its input, not {params['weight_on']!r}")
+        self.input_weight = params.get("weight_on", "output") == "input"
         self.renorm_eps = float(params.get("renorm_eps", 0.0))
         self.shared_size = int(params.get("shared_size") or 0)
         self.always = -(-self.shared_size // self.inter) if self.shared_size else 0
@@ -194,7 +200,8 @@ class MixtureOfExperts(FeedForward):
                 renormalize=self.renormalize, activation=self.activation, chosen=chosen, weight=weight, scratch=scratch,
                 act=act, rows=rows, xs=xs, ys=ys, gated=self.gated, correction=self.correction, identity=self.identity,
                 always=self.always, route_scale=self.route_scale, renorm_eps=self.renorm_eps, logit_scores=self.logit_scores,
-                always_gate=self.shared_gate, unit_limit=self.unit_limit, unit_slope=self.unit_slope)
+                always_gate=self.shared_gate, unit_limit=self.unit_limit, unit_slope=self.unit_slope,
+                input_weight=self.input_weight)
         if residual is None:
             return rows, self.slots
         ops.add_rows(rows, self.slots, residual)

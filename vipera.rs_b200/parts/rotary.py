@@ -111,6 +111,46 @@ def rotary_tables(head_dim: int, theta: float, max_positions: int, device, scali
     return tables
 
 
+def log_factor_table(coef: float, every: float, max_positions: int, device) -> _Tables:
+    """float32 [max_positions]: ``1 + coef ln(floor((p + 1) / every) + 1)`` for position p, formed in 64-bit
+    and rounded once."""
+    key = ("log_factor", float(coef), float(every), int(max_positions), str(device))
+    cached = _TABLES.get(key)
+    if cached is None:
+        position = torch.arange(int(max_positions), dtype=torch.float64)
+        values = 1.0 + float(coef) * torch.log(torch.floor((position + 1.0) / float(every)) + 1.0)
+        cached = _TABLES[key] = _Tables(values.to(torch.float32).contiguous().to(device), None)
+    return cached
+
+
+class QueryFactor:
+    """A number per position that multiplies the queries there: ``1 + coef ln(floor((p + 1) / every) + 1)``.
+    Attention owns one (params ``query_temperature`` = ``{"coef", "every"}``); its table is sized like a rotation's."""
+
+    def __init__(self, params, max_positions: int, device):
+        self.coef, self.every = float(params["coef"]), float(params["every"])
+        if not self.every > 0:
+            raise InvalidArgumentError(f"query_temperature: every must be positive, not {self.every}")
+        self.max_positions, self.device = int(max_positions), device
+        self.reach = None
+        self._table = None
+
+    def prepare(self, max_positions: int) -> None:
+        reach = min(self.max_positions, int(max_positions))
+        if self.reach is not None and reach <= self.reach:
+            return
+        self.reach = reach
+        if self._table is not None:   # a table in use moves: graphs that captured its address are stale
+            self._table = None
+            ops.buffer_generation += 1
+
+    def table(self):
+        if self._table is None:
+            self.reach = self.reach or self.max_positions
+            self._table = log_factor_table(self.coef, self.every, self.reach, self.device)
+        return self._table.pair[0]
+
+
 class RopeNeox(PositionEncoding):
     """params: ``head_dim``, ``theta``, ``max_positions`` and, optionally, ``rotary_dims`` (only
     the first that many values of a head turn, value i with value i + rotary_dims/2; default: the
