@@ -885,6 +885,95 @@ def nuvezen_decode_bytes(config, batch, history, element=2):
     return {"weights": weights * element, "state": 0, "cache": int(cache)}
 
 
+# ---------------------------------------------------------------------------------------
+# --design zugutar: the Zugutar design beside the Qwen2 decoder (or another design) at equal sizes
+# ---------------------------------------------------------------------------------------
+def zugutar_config(width, heads, kv_heads, ff, layers, vocab, *_unused, experts=16, top=4):
+    """`layers` layer runs: the last three of `layers` - 3 layers run twice.  Every fourth layer is attention
+    without positions (heads of 128, a gate per value), the others are two mixers side by side: softmax attention
+    (heads of 128, a norm per head, all values turning) and Mamba-2 with the width in channels (heads of 64, 128
+    states, 8 groups).  Every layer has a mixture of `experts` gated units of which a token uses `top`, beside a
+    gated shared unit, each a fifth of the dense inner size."""
+    piece = ff // (top + 1) // 16 * 16
+    moe = {"kind": "moe", "expert": {"ff": piece}, "shared": {"ff": piece}, "router": {"experts": experts, "top": top}}
+    sizes = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    attention = {**sizes, "q_temp": {"coef": 0.1, "every": 8192}}
+    both = {"left": {**sizes, "rot": {"dims": 128, "base": 500000.0}},
+            "right": {"heads": width // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}}
+    own = layers - 3
+    return {"architecture": "Zugutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "loop": {"start": own - 3, "stop": own, "times": 2},
+            "layers": [{"type": "attention", "mixer": attention, "mlp": moe} if index % 4 == 3 else
+                       {"type": "parallel", "mixer": both, "mlp": moe} for index in range(own)]}
+
+
+def _zugutar_runs(config):
+    loop = config["loop"]
+    inside = config["layers"][loop["start"]:loop["stop"]]
+    return config["layers"][:loop["start"]] + inside * loop["times"] + config["layers"][loop["stop"]:]
+
+
+def zugutar_work(config, tokens, chunk=128):
+    """Floating-point operations of a prompt of `tokens` tokens by class of kernel (as fasolorn_work); the
+    recurrence as its chunked form has them: scores within a chunk once per group, weighted sums, the read of the
+    state and its update."""
+    width = config["width"]
+    flops = {"proj": 2.0 * config["vocab"] * width, "attention": 0.0, "experts": 0.0, "recurrence": 0.0}
+    seen = tokens * (tokens + 1) // 2     # (query, key) pairs
+    for layer in _zugutar_runs(config):
+        m = layer["mixer"]
+        softmax = m if layer["type"] == "attention" else m["left"]
+        h, g, d, dv = softmax["heads"], softmax["kv_heads"], softmax["dim"], softmax["vdim"]
+        flops["proj"] += 2.0 * tokens * width * (h * d + g * (d + dv) + h * dv + (h * dv if softmax is m else h))
+        flops["attention"] += 2.0 * seen * h * (d + dv)
+        if softmax is not m:
+            r = m["right"]
+            inner, n = r["heads"] * r["vdim"], r["state"]
+            flops["proj"] += 2.0 * tokens * width * (3 * inner + 2 * r["groups"] * n + r["heads"])
+            flops["recurrence"] += 2.0 * tokens * (chunk / 2 * (r["groups"] * n + inner) + 2 * inner * n)
+        mlp = layer["mlp"]
+        inner = mlp["router"]["top"] * mlp["expert"]["ff"] + mlp["shared"]["ff"]
+        flops["experts"] += 2.0 * tokens * (3 * width * inner + (mlp["router"]["experts"] + 1) * width)
+    return flops
+
+
+def zugutar_prefill_bytes(config, tokens, chunk=128):
+    """What the recurrences of a prompt must move: x, B and C once in 16-bit, step sizes and gates in 32-bit,
+    outputs out in 32-bit and back for their norm, out in 16-bit; the 32-bit states at the chunks' starts four
+    times."""
+    moved = 0
+    for layer in _zugutar_runs(config):
+        if layer["type"] != "attention":
+            r = layer["mixer"]["right"]
+            inner = r["heads"] * r["vdim"]
+            moved += tokens * ((inner + 2 * r["groups"] * r["state"]) * 2 + r["heads"] * 4 + inner * (4 + 4 + 4 + 2))
+            moved += 4 * (-(-tokens // chunk)) * inner * r["state"] * 4
+    return moved
+
+
+def zugutar_decode_bytes(config, batch, history, element=2):
+    """What one decode step must move: every run's matrices that a token of the batch can use (all experts once
+    the batch's choices cover them), keys and values, and the recurrences' states read and written."""
+    width = config["width"]
+    weights, cache, state = config["vocab"] * width, 0, 0
+    for layer in _zugutar_runs(config):
+        m = layer["mixer"]
+        softmax = m if layer["type"] == "attention" else m["left"]
+        h, g, d, dv = softmax["heads"], softmax["kv_heads"], softmax["dim"], softmax["vdim"]
+        weights += width * (h * d + g * (d + dv) + h * dv + (h * dv if softmax is m else h))
+        cache += batch * history * g * (d + dv) * element
+        if softmax is not m:
+            r = m["right"]
+            inner = r["heads"] * r["vdim"]
+            weights += width * (3 * inner + 2 * r["groups"] * r["state"] + r["heads"])
+            state += 2 * batch * 4 * (inner * r["state"] + (inner + 2 * r["groups"] * r["state"]) * (r["conv"] - 1))
+        router = layer["mlp"]["router"]
+        used = min(router["experts"], batch * router["top"])
+        weights += 3 * width * (used * layer["mlp"]["expert"]["ff"] + layer["mlp"]["shared"]["ff"])
+        weights += (router["experts"] + 1) * width * 2     # the router's matrix is 32-bit
+    return {"weights": weights * element, "state": state, "cache": int(cache)}
+
+
 DESIGNS = {
     "nobupel": (lambda *sizes: nobupel_config(*sizes), lambda config, tokens: nobupel_work(config, tokens),
                 lambda config, batch, history: nobupel_decode_bytes(config, batch, history)),
@@ -896,6 +985,8 @@ DESIGNS = {
                  lambda config, batch, history: fasolorn_decode_bytes(config, batch, history)),
     "nuvezen": (lambda *sizes: nuvezen_config(*sizes), lambda config, tokens: nuvezen_work(config, tokens),
                 lambda config, batch, history: nuvezen_decode_bytes(config, batch, history)),
+    "zugutar": (lambda *sizes: zugutar_config(*sizes), lambda config, tokens: zugutar_work(config, tokens),
+                lambda config, batch, history: zugutar_decode_bytes(config, batch, history)),
 }
 
 
@@ -966,8 +1057,8 @@ def measure_design(args, peaks, peak_source):
                 out["prefill_frac_by_class"] = {
                     k: round(v / (out["prefill_ms_by_class"][k] * 1e-3) / (peaks["bf16_tflops"] * 1e12), 4)
                     for k, v in work.items() if out["prefill_ms_by_class"].get(k)}
-                if label == "gusolix" and out["prefill_ms_by_class"].get("recurrence"):
-                    moved = gusolix_prefill_bytes(config, tokens)
+                if label in ("gusolix", "zugutar") and out["prefill_ms_by_class"].get("recurrence"):
+                    moved = (gusolix_prefill_bytes if label == "gusolix" else zugutar_prefill_bytes)(config, tokens)
                     out["prefill_recurrence_hbm_frac"] = round(
                         moved / (out["prefill_ms_by_class"]["recurrence"] * 1e-3) / 1e9 / peaks["hbm_gbs"], 4)
             else:

@@ -239,8 +239,11 @@ def test_the_recurrence(name, form):
     y_d = torch.full((tokens, inner), float("nan"), device=DEV)
     out = torch.full((tokens, inner), float("nan"), dtype=dtype, device=DEV)
     jobs = ops.mamba2_jobs(tokens, entries)
-    chunks = (torch.full((jobs, heads * n * size), float("nan"), device=DEV), torch.full((jobs, heads), float("nan"), device=DEV)) \
-        if form == "chunks" else None
+    chunks = None
+    if form == "chunks":
+        chunks = (torch.full((jobs, heads * n * size), float("nan"), device=DEV),
+                  torch.full((jobs, 2 * heads * n * size), float("nan"), dtype=torch.bfloat16, device=DEV),
+                  torch.full((jobs, heads), float("nan"), device=DEV))
     ops.mamba2(xbc.to(DEV), proj.to(DEV), z_off=z_off, dt_off=dt_off, heads=heads, vdim=size, groups=groups, states=n,
                dt_bias=dt_bias.to(DEV), a=a.to(DEV), d=d.to(DEV), state=state, entry_starts=starts.to(DEV), state_slots=slots.to(DEV),
                fresh=fresh.to(DEV), num_entries=entries, any_single=1 in counts, y=y_d, norm_weight=weight.to(DEV),
@@ -275,8 +278,10 @@ def test_heads_that_share_their_scores(heads, groups, blocks, monkeypatch):
         state, y = start.clone(), torch.full((tokens, inner), float("nan"), device=DEV)
         out = torch.full((tokens, inner), float("nan"), dtype=torch.bfloat16, device=DEV)
         jobs = ops.mamba2_jobs(tokens, 2)
-        ops.mamba2(xbc, proj, state=state, y=y, out=out, chunks=(torch.empty(jobs, heads * n * size, device=DEV),
-                                                               torch.empty(jobs, heads, device=DEV)), **args)
+        ops.mamba2(xbc, proj, state=state, y=y, out=out, **args,
+                   chunks=(torch.empty(jobs, heads * n * size, device=DEV),
+                           torch.empty(jobs, 2 * heads * n * size, dtype=torch.bfloat16, device=DEV),
+                           torch.empty(jobs, heads, device=DEV)))
         results.append((state, y, out))
     assert all(torch.equal(one, other) and torch.isfinite(one.float()).all() for one, other in zip(*results))
 

@@ -55,8 +55,9 @@ struct Mamba2Params {
   float* y;                 // [tokens, heads * vdim] before gate and norm
   const float* norm_weight; // [heads * vdim]
   void* out;                // [tokens, heads * vdim] the run's type
-  float* chunk_state;       // [jobs, heads, state, vdim]   (chunks only)
-  float* chunk_decay;       // [jobs, heads] l_L
+  float* chunk_state;       // [jobs, heads, state, vdim] a chunk's own sum   (chunks only)
+  void* chunk_start;        // [jobs, heads, 2, state, vdim] bfloat16: high, then low halves of the state at a chunk's start
+  float* chunk_decay;       // [jobs, heads] l_L / ln 2
   int heads, vdim, groups, states, norm_groups, num_entries, num_tokens, num_jobs;
   int heads_per_block;      // chunks: heads of one group a block works on
   int single_only;          // walk: entries of other than one token are left out
@@ -232,7 +233,7 @@ __device__ __forceinline__ void find_chunk(const int* __restrict__ entry_starts,
 }
 
 // Step sizes and running sums of log decays of a chunk's tokens (a warp; four tokens a lane).
-// dt[t] and l[t] = a (dt[0] + .. + dt[t]); tokens past the chunk's end have dt = 0.
+// dt[t] and l[t] = a (dt[0] + .. + dt[t]) / ln 2; tokens past the chunk's end have dt = 0.
 __device__ __forceinline__ void chunk_decays(const Mamba2Params& p, int begin, int len, int h, float* dt, float* l) {
   const int lane = threadIdx.x & 31;
   float own[4], sum = 0.0f;
@@ -250,7 +251,7 @@ __device__ __forceinline__ void chunk_decays(const Mamba2Params& p, int begin, i
     if (lane >= offset) upto += other;
   }
   float running = upto - sum;
-  const float a = p.a[h];
+  const float a = p.a[h] * 1.4426950408889634f;
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     running += own[j];
@@ -283,18 +284,25 @@ __device__ __forceinline__ void split_pair(float u, float v, uint32_t& high, uin
   low = *reinterpret_cast<const uint32_t*>(&r);
 }
 
+// 16 bytes from global to shared memory without a register in between, or 16 zero bytes.
+__device__ __forceinline__ void copy_16(void* dst, const void* src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(shared_address(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void copies_wait() {
+  asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory");
+}
+
 // Rows of bfloat16 from global memory into shared memory rows of `stride` values: `width` values of `rows`
 // rows, zeros up to `padded` values and `total` rows.  `vectors`: every row starts on 16 bytes and width is
-// a multiple of eight.
+// a multiple of eight; the copies are then on their way until copies_wait().
 __device__ __forceinline__ void load_rows(__nv_bfloat16* dst, int stride, const __nv_bfloat16* src, long long src_stride, int rows,
                                           int total, int width, int padded, bool vectors) {
   if (vectors) {
     const int pieces = padded / 8;
     for (int i = threadIdx.x; i < total * pieces; i += kThreads) {
       const int r = i / pieces, c = (i % pieces) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < rows && c < width) v = *reinterpret_cast<const uint4*>(src + r * src_stride + c);
-      *reinterpret_cast<uint4*>(dst + r * stride + c) = v;
+      const bool live = r < rows && c < width;
+      copy_16(dst + r * stride + c, live ? src + r * src_stride + c : src, live);
     }
   } else {
     for (int i = threadIdx.x; i < total * padded; i += kThreads) {
@@ -361,7 +369,7 @@ mamba2_parts_kernel(const Mamba2Params p) {
         if (t < len && c < cols) {
           const uint4 v = *reinterpret_cast<const uint4*>(x + t * p.xbc_width + c);
           const __nv_bfloat162* pairs = reinterpret_cast<const __nv_bfloat162*>(&v);
-          const float w = expf(last - l_s[t]) * dt_s[t];
+          const float w = exp2f(last - l_s[t]) * dt_s[t];
           uint32_t* hp = reinterpret_cast<uint32_t*>(&high);
           uint32_t* lp = reinterpret_cast<uint32_t*>(&low);
 #pragma unroll
@@ -377,13 +385,14 @@ mamba2_parts_kernel(const Mamba2Params p) {
       for (int item = threadIdx.x; item < steps * 16 * kCols; item += kThreads) {
         const int t = item / kCols, c = item % kCols;
         float v = 0.0f;
-        if (t < len && c < cols) v = expf(last - l_s[t]) * dt_s[t] * __bfloat162float(x[t * p.xbc_width + c]);
+        if (t < len && c < cols) v = exp2f(last - l_s[t]) * dt_s[t] * __bfloat162float(x[t * p.xbc_width + c]);
         const __nv_bfloat16 high = __float2bfloat16_rn(v);
         Xh[t * kXStride + c] = high;
         Xl[t * kXStride + c] = __float2bfloat16_rn(v - __bfloat162float(high));
       }
     }
     if (threadIdx.x == 0 && blockIdx.z == 0) p.chunk_decay[job_base + h] = last;
+    copies_wait();   // b, ahead of the first head's product
     __syncthreads();
     float* E = p.chunk_state + (job_base + h) * static_cast<size_t>(p.states) * p.vdim;
     // a warp's job: sixteen rows of the state by 32 columns
@@ -430,7 +439,7 @@ mamba2_parts_kernel(const Mamba2Params p) {
 }
 
 // grid: (pieces of a head's state, heads, entries).  A thread VEC neighbouring values, the entry's chunks
-// in order, four chunks' sums asked for together: leaves the state at each chunk's start in its place.
+// in order, eight chunks' sums asked for together: leaves the state at each chunk's start as two halves.
 template <int VEC>
 __global__ void __launch_bounds__(kThreads)
 mamba2_carry_kernel(const Mamba2Params p) {
@@ -457,16 +466,26 @@ mamba2_carry_kernel(const Mamba2Params p) {
       v[0] = *at;
     }
   };
-  auto store = [](float* at, const float (&v)[VEC]) {
-    if constexpr (VEC == 4) *reinterpret_cast<float4*>(at) = make_float4(v[0], v[1], v[2], v[3]);
-    else *at = v[0];
+  auto store_halves = [&](__nv_bfloat16* at, const float (&v)[VEC]) {
+    if constexpr (VEC == 4) {
+      uint2 high, low;
+      split_pair(v[0], v[1], high.x, low.x);
+      split_pair(v[2], v[3], high.y, low.y);
+      *reinterpret_cast<uint2*>(at) = high;
+      *reinterpret_cast<uint2*>(at + head_size) = low;
+    } else {
+      const __nv_bfloat16 high = __float2bfloat16_rn(v[0]);
+      at[0] = high;
+      at[head_size] = __float2bfloat16_rn(v[0] - __bfloat162float(high));
+    }
   };
   float s[VEC];
 #pragma unroll
   for (int e = 0; e < VEC; ++e) s[e] = 0.0f;
   if (!fresh) load(s, own);
   const size_t job_stride = static_cast<size_t>(p.heads) * head_size;
-  float* E = p.chunk_state + (static_cast<size_t>(job0) * p.heads + h) * head_size + index;
+  const float* E = p.chunk_state + (static_cast<size_t>(job0) * p.heads + h) * head_size + index;
+  __nv_bfloat16* starts = static_cast<__nv_bfloat16*>(p.chunk_start) + (static_cast<size_t>(job0) * p.heads + h) * 2 * head_size + index;
   const float* decay = p.chunk_decay + static_cast<size_t>(job0) * p.heads + h;
   for (int c0 = 0; c0 < chunks; c0 += 8) {
     float sums[8][VEC], l[8];
@@ -480,17 +499,18 @@ mamba2_carry_kernel(const Mamba2Params p) {
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       if (c0 + j >= chunks) break;
-      store(E + (c0 + j) * job_stride, s);
-      const float keep = expf(l[j]);
+      store_halves(starts + (c0 + j) * 2 * job_stride, s);
+      const float keep = exp2f(l[j]);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) s[e] = fmaf(keep, s[e], sums[j][e]);
     }
   }
-  store(own, s);
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(own) = make_float4(s[0], s[1], s[2], s[3]);
+  else *own = s[0];
 }
 
 // grid: (jobs, heads / heads_per_block, column tiles).  A warp owns sixteen tokens of the chunk.
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, 2)
 mamba2_outputs_kernel(const Mamba2Params p) {
   extern __shared__ __align__(16) unsigned char raw[];
   __shared__ int info[3];
@@ -517,6 +537,7 @@ mamba2_outputs_kernel(const Mamba2Params p) {
   const size_t c_off = b_off + static_cast<size_t>(p.groups) * p.states;
   load_rows(Bs, bs, rows + b_off, p.xbc_width, len, steps * 16, p.states, np, rows_on_16_bytes(p, b_off, p.states));
   load_rows(Cs, bs, rows + c_off, p.xbc_width, len, steps * 16, p.states, np, rows_on_16_bytes(p, c_off, p.states));
+  copies_wait();
   __syncthreads();
   // the scores of the warp's tokens with every token up to them: once for all heads of the block
   const bool live = warp * 16 < len;
@@ -546,27 +567,13 @@ mamba2_outputs_kernel(const Mamba2Params p) {
     if (warp == 0) chunk_decays(p, begin, len, h, dt_s, l_s);
     const size_t x_off = static_cast<size_t>(h) * p.vdim + col0;
     load_rows(Xs, kXStride, rows + x_off, p.xbc_width, len, steps * 16, cols, kCols, rows_on_16_bytes(p, x_off, cols));
-    const float* S0 = p.chunk_state + (static_cast<size_t>(blockIdx.x) * p.heads + h) * static_cast<size_t>(p.states) * p.vdim + col0;
-    if ((p.vdim & 3) == 0) {
-      for (int item = threadIdx.x; item < np * (kCols / 4); item += kThreads) {
-        const int n = item / (kCols / 4), c = (item % (kCols / 4)) * 4;
-        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        if (n < p.states && c < cols) v = *reinterpret_cast<const float4*>(S0 + static_cast<size_t>(n) * p.vdim + c);
-        uint2 high, low;
-        split_pair(v.x, v.y, high.x, low.x);
-        split_pair(v.z, v.w, high.y, low.y);
-        *reinterpret_cast<uint2*>(Sh + n * kXStride + c) = high;
-        *reinterpret_cast<uint2*>(Sl + n * kXStride + c) = low;
-      }
-    } else {
-      for (int item = threadIdx.x; item < np * kCols; item += kThreads) {
-        const int n = item / kCols, c = item % kCols;
-        const float v = (n < p.states && c < cols) ? S0[static_cast<size_t>(n) * p.vdim + c] : 0.0f;
-        const __nv_bfloat16 high = __float2bfloat16_rn(v);
-        Sh[n * kXStride + c] = high;
-        Sl[n * kXStride + c] = __float2bfloat16_rn(v - __bfloat162float(high));
-      }
-    }
+    const size_t head_size = static_cast<size_t>(p.states) * p.vdim;
+    const __nv_bfloat16* S0 = static_cast<const __nv_bfloat16*>(p.chunk_start) +
+                              (static_cast<size_t>(blockIdx.x) * p.heads + h) * 2 * head_size + col0;
+    const bool whole = p.vdim % 8 == 0 && (reinterpret_cast<uintptr_t>(p.chunk_start) & 15) == 0;
+    load_rows(Sh, kXStride, S0, p.vdim, p.states, np, cols, kCols, whole);
+    load_rows(Sl, kXStride, S0 + head_size, p.vdim, p.states, np, cols, kCols, whole);
+    copies_wait();
     __syncthreads();
     if (!live) continue;
     float y[kCols / 8][4];
@@ -591,7 +598,7 @@ mamba2_outputs_kernel(const Mamba2Params p) {
       }
     }
     const float l_first = l_s[row0], l_second = l_s[row0 + 8];
-    const float from_start[2] = {expf(l_first), expf(l_second)};
+    const float from_start[2] = {exp2f(l_first), exp2f(l_second)};
 #pragma unroll
     for (int nt = 0; nt < kCols / 8; ++nt)
 #pragma unroll
@@ -611,7 +618,7 @@ mamba2_outputs_kernel(const Mamba2Params p) {
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           const int col = nt * 8 + 2 * (lane & 3) + j;
-          w[j] = col <= row ? scores[nt][e + j] * (expf(l_row - l_s[col]) * dt_s[col]) : 0.0f;
+          w[j] = col <= row ? scores[nt][e + j] * (exp2f(l_row - l_s[col]) * dt_s[col]) : 0.0f;
         }
         split_pair(w[0], w[1], high[part], low[part]);
       }
@@ -694,6 +701,72 @@ mamba2_finish_kernel(const Mamba2Params p) {
   }
 }
 
+// The same for parts of up to 128 * PIECES values that are whole vectors: a warp a part, the part in registers
+// between its passes.
+template <typename T, int PIECES>
+__global__ void __launch_bounds__(kThreads)
+mamba2_finish_rows_kernel(const Mamba2Params p) {
+  pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long job = static_cast<long long>(blockIdx.x) * (kThreads / 32) + warp;
+  const int width = p.heads * p.vdim, size = width / p.norm_groups;
+  if (job >= static_cast<long long>(p.num_tokens) * p.norm_groups) return;
+  const size_t t = job / p.norm_groups;
+  const int first = static_cast<int>(job % p.norm_groups) * size;
+  pdl_wait();
+  const float* y = p.y + t * width + first;
+  const float* z = p.proj + t * p.proj_width + p.z_off + first;
+  float4 kept[PIECES], gate[PIECES];
+#pragma unroll
+  for (int j = 0; j < PIECES; ++j) {
+    const int i = 4 * (lane + 32 * j);
+    kept[j] = gate[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (i < size) {
+      kept[j] = *reinterpret_cast<const float4*>(y + i);
+      gate[j] = *reinterpret_cast<const float4*>(z + i);
+    }
+  }
+  auto silu = [](float v) { return v / (1.0f + expf(-v)); };
+  float sum = 0.0f;
+#pragma unroll
+  for (int j = 0; j < PIECES; ++j) {
+    kept[j].x *= silu(gate[j].x), kept[j].y *= silu(gate[j].y), kept[j].z *= silu(gate[j].z), kept[j].w *= silu(gate[j].w);
+    sum = fmaf(kept[j].x, kept[j].x, sum), sum = fmaf(kept[j].y, kept[j].y, sum);
+    sum = fmaf(kept[j].z, kept[j].z, sum), sum = fmaf(kept[j].w, kept[j].w, sum);
+  }
+  const float inverse = 1.0f / sqrtf(warp_sum(sum) / static_cast<float>(size) + p.eps);
+  T* out = static_cast<T*>(p.out) + t * width + first;
+#pragma unroll
+  for (int j = 0; j < PIECES; ++j) {
+    const int i = 4 * (lane + 32 * j);
+    if (i >= size) continue;
+    const float4 w = *reinterpret_cast<const float4*>(p.norm_weight + first + i);
+    const float v[4] = {kept[j].x * inverse * w.x, kept[j].y * inverse * w.y, kept[j].z * inverse * w.z, kept[j].w * inverse * w.w};
+    if constexpr (sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(out + i) = make_float4(v[0], v[1], v[2], v[3]);
+    } else {
+      __nv_bfloat162 pair[2] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3])};
+      *reinterpret_cast<uint2*>(out + i) = *reinterpret_cast<const uint2*>(pair);
+    }
+  }
+}
+
+template <typename T>
+static int launch_finish(const Mamba2Params& p, cudaStream_t s) {
+  const int size = p.heads * p.vdim / p.norm_groups;
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(p.y) | reinterpret_cast<uintptr_t>(p.proj) | reinterpret_cast<uintptr_t>(p.out) |
+                          reinterpret_cast<uintptr_t>(p.norm_weight);
+  if (size % 4 == 0 && size <= 1024 && p.proj_width % 4 == 0 && p.z_off % 4 == 0 && (bases & 15) == 0) {
+    const long long jobs = static_cast<long long>(p.num_tokens) * p.norm_groups;
+    const unsigned grid = static_cast<unsigned>((jobs + kThreads / 32 - 1) / (kThreads / 32));
+    if (size <= 256) return vipera_launch(mamba2_finish_rows_kernel<T, 2>, grid, kThreads, 0, s, p);
+    if (size <= 512) return vipera_launch(mamba2_finish_rows_kernel<T, 4>, grid, kThreads, 0, s, p);
+    return vipera_launch(mamba2_finish_rows_kernel<T, 8>, grid, kThreads, 0, s, p);
+  }
+  const int threads = size >= 256 ? 256 : (size + 31) / 32 * 32;
+  return vipera_launch(mamba2_finish_kernel<T>, dim3(p.num_tokens, p.norm_groups), threads, 0, s, p);
+}
+
 // ---------------------------------------------------------------------------------------
 template <typename T, int ROWS>
 static int launch_walk(const Mamba2Params& p, cudaStream_t s) {
@@ -724,7 +797,7 @@ static int launch_chunks(const Mamba2Params& p, cudaStream_t s) {
   int status = vipera_launch(mamba2_parts_kernel, grid, kThreads, parts_shared(p.states), s, p);
   if (status) return status;
   const size_t head_size = static_cast<size_t>(p.states) * p.vdim;
-  const bool four = head_size % 4 == 0 && ((reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(p.chunk_state)) & 15) == 0;
+  const bool four = head_size % 4 == 0 && ((reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(p.chunk_state) | reinterpret_cast<uintptr_t>(p.chunk_start)) & 15) == 0;
   const size_t per_block = static_cast<size_t>(kThreads) * (four ? 4 : 1);
   const dim3 carry_grid(static_cast<unsigned>((head_size + per_block - 1) / per_block), p.heads, p.num_entries);
   status = four ? vipera_launch(mamba2_carry_kernel<4>, carry_grid, kThreads, 0, s, p)
@@ -743,7 +816,7 @@ VIPERA_API int vipera_mamba2(const Mamba2Params* params, int dtype, int any_sing
       p.heads % p.groups || p.norm_groups <= 0 || p.norm_groups > 65535 || (p.heads * p.vdim) % p.norm_groups || p.num_entries > 65535)
     return VIPERA_BAD_SHAPE;
   const bool chunked = p.num_jobs > 0;
-  if (chunked && (dtype != VIPERA_BF16 || !p.chunk_state || !p.chunk_decay || p.heads_per_block <= 0 ||
+  if (chunked && (dtype != VIPERA_BF16 || !p.chunk_state || !p.chunk_start || !p.chunk_decay || p.heads_per_block <= 0 ||
                   (p.heads / p.groups) % p.heads_per_block))
     return VIPERA_BAD_ARGUMENT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
@@ -757,11 +830,7 @@ VIPERA_API int vipera_mamba2(const Mamba2Params* params, int dtype, int any_sing
     else return VIPERA_BAD_DTYPE;
     if (status) return status;
   }
-  const int size = p.heads * p.vdim / p.norm_groups;
-  const int threads = size >= 256 ? 256 : (size + 31) / 32 * 32;
-  const dim3 grid(p.num_tokens, p.norm_groups);
-  if (dtype == VIPERA_F32) return vipera_launch(mamba2_finish_kernel<float>, grid, threads, 0, s, p);
-  return vipera_launch(mamba2_finish_kernel<__nv_bfloat16>, grid, threads, 0, s, p);
+  return dtype == VIPERA_F32 ? launch_finish<float>(p, s) : launch_finish<__nv_bfloat16>(p, s);
 }
 
 VIPERA_API int vipera_mamba2_params_size() { return static_cast<int>(sizeof(Mamba2Params)); }

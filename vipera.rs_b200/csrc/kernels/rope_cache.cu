@@ -436,6 +436,139 @@ head_rows_kernel(const HeadRowsParams p) {
   }
 }
 
+// The same where everything is whole vectors of four (heads of up to 128 * PIECES values): a lane holds
+// values 4 (lane + 32 j) .. + 3 of each of its warp's kHeadJobs heads, whose loads are in flight together.
+constexpr int kHeadJobs = 2;
+
+template <typename T, int PIECES>
+__global__ void __launch_bounds__(kHeadWarps * 32)
+head_rows_vector_kernel(const HeadRowsParams p) {
+  __shared__ __align__(16) float rows[kHeadWarps][128 * PIECES];
+  pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x;
+  const int position = p.positions[t];
+  const int jobs = p.num_heads + 2 * p.num_kv_heads;
+  const int job0 = (blockIdx.y * kHeadWarps + warp) * kHeadJobs;
+  if (job0 >= jobs) return;
+  size_t place = 0;
+  bool stored = false;
+  if (p.write_cache) {
+    const int page = p.block_table[static_cast<size_t>(p.token_entry[t]) * p.table_width + position / p.page_size];
+    stored = page >= 0;
+    place = static_cast<size_t>(max(page, 0)) * p.page_size + position % p.page_size;
+  }
+  const float factor = p.q_factor ? p.q_factor[position] : 1.0f;
+  const int half = p.rot_dims >> 1;
+  const bool turns = p.style != ROPE_NONE && p.rot_dims > 0;
+  pdl_wait();
+  const float* row = p.qkv + static_cast<long long>(t) * p.row_stride;
+  float4 x[kHeadJobs][PIECES];
+#pragma unroll
+  for (int n = 0; n < kHeadJobs; ++n) {
+    const int job = job0 + n;
+    const bool is_v = job >= p.num_heads + p.num_kv_heads;
+    const int size = job >= jobs ? 0 : (is_v ? p.value_dim : p.head_dim);
+    const float* src = row + (is_v ? (p.num_heads + p.num_kv_heads) * p.head_dim + (job - p.num_heads - p.num_kv_heads) * p.value_dim
+                                   : job * p.head_dim);
+#pragma unroll
+    for (int j = 0; j < PIECES; ++j) {
+      const int e = 4 * (lane + 32 * j);
+      x[n][j] = e < size ? *reinterpret_cast<const float4*>(src + e) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < kHeadJobs; ++n) {
+    const int job = job0 + n;
+    if (job >= jobs) break;
+    const bool is_q = job < p.num_heads, is_v = job >= p.num_heads + p.num_kv_heads;
+    const int size = is_v ? p.value_dim : p.head_dim;
+    const float* gain = is_v ? nullptr : (is_q ? p.q_norm : p.k_norm);
+    if (gain) {
+      float sum = 0.0f;
+#pragma unroll
+      for (int j = 0; j < PIECES; ++j)
+        sum += x[n][j].x * x[n][j].x + x[n][j].y * x[n][j].y + x[n][j].z * x[n][j].z + x[n][j].w * x[n][j].w;
+      const float inverse = 1.0f / sqrtf(warp_sum(sum) / static_cast<float>(size) + p.eps);
+#pragma unroll
+      for (int j = 0; j < PIECES; ++j) {
+        const int e = 4 * (lane + 32 * j);
+        if (e < size) {
+          const float4 g = *reinterpret_cast<const float4*>(gain + e);
+          x[n][j] = make_float4(x[n][j].x * inverse * g.x, x[n][j].y * inverse * g.y, x[n][j].z * inverse * g.z, x[n][j].w * inverse * g.w);
+        }
+      }
+    }
+    if (turns && !is_v) {
+      const float* cos_row = p.cos_table + static_cast<size_t>(position) * half;
+      const float* sin_row = p.sin_table + static_cast<size_t>(position) * half;
+      if (p.style == ROPE_INTERLEAVED) {
+#pragma unroll
+        for (int j = 0; j < PIECES; ++j) {
+          const int e = 4 * (lane + 32 * j);
+          if (e < p.rot_dims) {
+            const float2 c = *reinterpret_cast<const float2*>(cos_row + e / 2), s = *reinterpret_cast<const float2*>(sin_row + e / 2);
+            const float4 v = x[n][j];
+            x[n][j] = make_float4(v.x * c.x - v.y * s.x, v.y * c.x + v.x * s.x, v.z * c.y - v.w * s.y, v.w * c.y + v.z * s.y);
+          }
+        }
+      } else {
+        // a value's partner belongs to another lane
+        __syncwarp();
+#pragma unroll
+        for (int j = 0; j < PIECES; ++j)
+          if (4 * (lane + 32 * j) < p.rot_dims) *reinterpret_cast<float4*>(&rows[warp][4 * (lane + 32 * j)]) = x[n][j];
+        __syncwarp();
+#pragma unroll
+        for (int j = 0; j < PIECES; ++j) {
+          const int e = 4 * (lane + 32 * j);
+          if (e < p.rot_dims) {
+            const bool second = e >= half;
+            const int i = second ? e - half : e;
+            const float4 o = *reinterpret_cast<const float4*>(&rows[warp][second ? e - half : e + half]);
+            const float4 c = *reinterpret_cast<const float4*>(cos_row + i);
+            float4 s = *reinterpret_cast<const float4*>(sin_row + i);
+            if (!second) s = make_float4(-s.x, -s.y, -s.z, -s.w);
+            const float4 v = x[n][j];
+            x[n][j] = make_float4(v.x * c.x + o.x * s.x, v.y * c.y + o.y * s.y, v.z * c.z + o.z * s.z, v.w * c.w + o.w * s.w);
+          }
+        }
+      }
+    }
+    T* dst;
+    if (is_q) dst = static_cast<T*>(p.q_out) + (static_cast<size_t>(t) * p.num_heads + job) * p.head_dim;
+    else if (!stored) continue;
+    else if (is_v) dst = static_cast<T*>(p.v_pool) + (place * p.num_kv_heads + (job - p.num_heads - p.num_kv_heads)) * p.value_dim;
+    else dst = static_cast<T*>(p.k_pool) + (place * p.num_kv_heads + (job - p.num_heads)) * p.head_dim;
+    const float f = is_q ? factor : 1.0f;
+#pragma unroll
+    for (int j = 0; j < PIECES; ++j) {
+      const int e = 4 * (lane + 32 * j);
+      if (e >= size) continue;
+      const float4 v = x[n][j];
+      store_pair(dst + e, v.x * f, v.y * f);
+      store_pair(dst + e + 2, v.z * f, v.w * f);
+    }
+  }
+}
+
+template <typename T>
+static int launch_head_rows(const HeadRowsParams& p, cudaStream_t s) {
+  const int jobs = p.num_heads + 2 * p.num_kv_heads;
+  const bool turns = p.style != ROPE_NONE && p.rot_dims > 0;
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(p.qkv) | reinterpret_cast<uintptr_t>(p.q_out) | reinterpret_cast<uintptr_t>(p.q_norm) |
+                          reinterpret_cast<uintptr_t>(p.k_norm) | reinterpret_cast<uintptr_t>(p.k_pool) | reinterpret_cast<uintptr_t>(p.v_pool) |
+                          (turns ? reinterpret_cast<uintptr_t>(p.cos_table) | reinterpret_cast<uintptr_t>(p.sin_table) : 0);
+  const bool vectors = p.head_dim % 4 == 0 && p.value_dim % 4 == 0 && p.row_stride % 4 == 0 && (bases & 15) == 0 &&
+                       (!turns || (p.style == ROPE_INTERLEAVED ? p.rot_dims % 4 == 0 : p.rot_dims % 8 == 0));
+  if (vectors) {
+    const dim3 grid(p.num_tokens, (jobs + kHeadWarps * kHeadJobs - 1) / (kHeadWarps * kHeadJobs));
+    if (p.head_dim <= 128 && p.value_dim <= 128) return vipera_launch(head_rows_vector_kernel<T, 1>, grid, kHeadWarps * 32, 0, s, p);
+    return vipera_launch(head_rows_vector_kernel<T, 2>, grid, kHeadWarps * 32, 0, s, p);
+  }
+  return vipera_launch(head_rows_kernel<T>, dim3(p.num_tokens, (jobs + kHeadWarps - 1) / kHeadWarps), kHeadWarps * 32, 0, s, p);
+}
+
 // dtype: the type of q_out and of the pools.
 VIPERA_API int vipera_head_rows(const HeadRowsParams* params, int dtype, void* stream) {
   const HeadRowsParams& p = *params;
@@ -446,10 +579,9 @@ VIPERA_API int vipera_head_rows(const HeadRowsParams* params, int dtype, void* s
   if (!p.qkv || !p.q_out || !p.positions) return VIPERA_BAD_ARGUMENT;
   if (p.style != ROPE_NONE && p.rot_dims > 0 && (!p.cos_table || !p.sin_table)) return VIPERA_BAD_ARGUMENT;
   if (p.write_cache && (!p.k_pool || !p.v_pool || !p.token_entry || !p.block_table || p.page_size <= 0)) return VIPERA_BAD_ARGUMENT;
-  const dim3 grid(p.num_tokens, (p.num_heads + 2 * p.num_kv_heads + kHeadWarps - 1) / kHeadWarps);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == VIPERA_F32) return vipera_launch(head_rows_kernel<float>, grid, kHeadWarps * 32, 0, s, p);
-  if (dtype == VIPERA_BF16) return vipera_launch(head_rows_kernel<__nv_bfloat16>, grid, kHeadWarps * 32, 0, s, p);
+  if (dtype == VIPERA_F32) return launch_head_rows<float>(p, s);
+  if (dtype == VIPERA_BF16) return launch_head_rows<__nv_bfloat16>(p, s);
   return VIPERA_BAD_DTYPE;
 }
 

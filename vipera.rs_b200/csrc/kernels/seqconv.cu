@@ -118,20 +118,26 @@ __global__ void __launch_bounds__(kConvThreads) causal_conv_kernel(const ConvPar
     }
     return;
   }
-  // segment job: tokens far enough into their entry to read only the step's own rows
+  // segment job: tokens far enough into their entry to read only the step's own rows.  The segment's inputs are
+  // asked for together and each is read once (rows in front of an entry's start are read and not used).
   const int begin = (job - p.num_entries) * kConvSegment;
-  const int end = min(begin + kConvSegment, p.num_tokens);
-  for (int t = begin; t < end; ++t) {
-    const int entry = p.token_entry[t];
-    const int index = t - p.entry_starts[entry];
-    if (index < taps - 1) continue;
+  float inputs[kConvSegment + MAXT - 1];
+#pragma unroll
+  for (int k = 0; k < kConvSegment + MAXT - 1; ++k) {
+    const int row = begin - (taps - 1) + k;
+    inputs[k] = (k < kConvSegment + taps - 1 && row >= 0 && row < p.num_tokens) ? p.x[static_cast<size_t>(row) * p.x_stride + c] : 0.0f;
+  }
+#pragma unroll
+  for (int i = 0; i < kConvSegment; ++i) {
+    const int t = begin + i;
+    if (t >= p.num_tokens) break;
+    if (t - p.entry_starts[p.token_entry[t]] < taps - 1) continue;
     float sum = 0.0f, current = 0.0f;
 #pragma unroll
     for (int j = 0; j < MAXT; ++j) {
       if (j < taps) {
-        const float value = p.x[static_cast<size_t>(t - (taps - 1) + j) * p.x_stride + c];
-        sum = fmaf(w[j], value, sum);
-        if (j == taps - 1) current = value;
+        sum = fmaf(w[j], inputs[i + j], sum);
+        if (j == taps - 1) current = inputs[i + j];
       }
     }
     conv_store<TO>(p, t, c, conv_finish(sum, current, p, bias));

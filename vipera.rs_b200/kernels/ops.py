@@ -1635,7 +1635,7 @@ class _Mamba2Params(ctypes.Structure):
         ("xbc", _c_void), ("xbc_width", ctypes.c_longlong), ("proj", _c_void), ("proj_width", ctypes.c_longlong),
         ("z_off", _c_int), ("dt_off", _c_int), ("dt_bias", _c_void), ("a", _c_void), ("d", _c_void), ("state", _c_void),
         ("entry_starts", _c_void), ("state_slots", _c_void), ("fresh", _c_void), ("y", _c_void), ("norm_weight", _c_void),
-        ("out", _c_void), ("chunk_state", _c_void), ("chunk_decay", _c_void),
+        ("out", _c_void), ("chunk_state", _c_void), ("chunk_start", _c_void), ("chunk_decay", _c_void),
         ("heads", _c_int), ("vdim", _c_int), ("groups", _c_int), ("states", _c_int), ("norm_groups", _c_int),
         ("num_entries", _c_int), ("num_tokens", _c_int), ("num_jobs", _c_int), ("heads_per_block", _c_int),
         ("single_only", _c_int), ("eps", _c_float),
@@ -1672,8 +1672,8 @@ def mamba2(xbc: torch.Tensor, proj: torch.Tensor, *, z_off: int, dt_off: int, he
     the gate z at column ``z_off`` and the raw step sizes at ``dt_off``; ``state`` float32 [slots, heads *
     states * vdim], read where an entry is not fresh and left as the entry's last token leaves it.  ``y``
     float32 [tokens, heads * vdim] is scratch; ``out`` (xbc's type) receives ``y * silu(z)`` divided by its root
-    mean square in ``norm_groups`` parts, times ``norm_weight``.  ``chunks`` (bfloat16: float32 tensors [jobs,
-    heads * states * vdim] and [jobs, heads], jobs >= mamba2_jobs(...)): entries of several tokens run as chunks
+    mean square in ``norm_groups`` parts, times ``norm_weight``.  ``chunks`` (bfloat16: tensors [jobs, heads *
+    states * vdim] float32, [jobs, 2 * heads * states * vdim] bfloat16 and [jobs, heads] float32, jobs >= mamba2_jobs(...)): entries of several tokens run as chunks
     side by side; ``any_single`` then says whether there are entries of one token beside them."""
     fn = _function("mamba2", "vipera_mamba2", [ctypes.POINTER(_Mamba2Params), _c_int, _c_int, _c_void])
     _check_struct("mamba2", "vipera_mamba2_params_size", _Mamba2Params)
@@ -1707,11 +1707,13 @@ def mamba2(xbc: torch.Tensor, proj: torch.Tensor, *, z_off: int, dt_off: int, he
     p.num_entries, p.num_tokens = int(num_entries), int(tokens)
     launched = 2
     if chunks is not None:
-        sums, decays = chunks
+        sums, halves, decays = chunks
         jobs = mamba2_jobs(tokens, num_entries)
-        if xbc.dtype != torch.bfloat16 or sums.numel() < jobs * heads * states * vdim or decays.numel() < jobs * heads:
+        if xbc.dtype != torch.bfloat16 or sums.numel() < jobs * heads * states * vdim or decays.numel() < jobs * heads or \
+                halves.numel() < 2 * jobs * heads * states * vdim:
             raise InvalidArgumentError("mamba2: the chunked form runs in bfloat16 and needs room for every chunk of the step")
         p.chunk_state, p.chunk_decay = _gpu(sums, "chunk states", torch.float32), _gpu(decays, "chunk decays", torch.float32)
+        p.chunk_start = _gpu(halves, "chunk starts", torch.bfloat16)
         p.num_jobs = jobs
         p.heads_per_block = mamba2_heads_per_block(jobs, int(heads), int(groups), int(vdim), sm_count(xbc.device))
         launched = 4 + int(bool(any_single))

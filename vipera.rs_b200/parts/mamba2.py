@@ -99,7 +99,7 @@ class Mamba2(Mixer):
         jobs = ops.mamba2_jobs(tokens, 1)
         return (tokens * ((inner + channels + heads) * 4 + channels * element_bytes + inner * (4 + element_bytes)
                           + int(params["hidden_size"]) * 4)
-                + jobs * heads * (int(params["state"]) * int(params["value_dim"]) + 1) * 4)
+                + jobs * heads * (2 * int(params["state"]) * int(params["value_dim"]) + 1) * 4)
 
     def forward(self, ctx, h, residual, cache, writes_cache):
         count, ws = ctx.num_tokens, ctx.workspace
@@ -113,6 +113,7 @@ class Mamba2(Mixer):
         if ctx.dtype == torch.bfloat16 and not ctx.all_single and count >= self.CHUNKED_FROM:
             jobs = ops.mamba2_jobs(count, ctx.num_entries)
             chunks = (ws.get("mamba2.chunk_state", (jobs, self.heads * self.state * self.vdim), torch.float32),
+                      ws.get("mamba2.chunk_start", (jobs, 2 * self.heads * self.state * self.vdim), torch.bfloat16),
                       ws.get("mamba2.chunk_decay", (jobs, self.heads), torch.float32))
         ops.mamba2(xbc, proj, z_off=0, dt_off=self.inner + self.channels, heads=self.heads, vdim=self.vdim,
                    groups=self.groups, states=self.state, dt_bias=self.dt_bias, a=self.a, d=self.d,
