@@ -16,6 +16,7 @@ from vipera_rs_b200 import errors
 from vipera_rs_b200.cache.pools import plan_groups
 from vipera_rs_b200.config import architecture_of
 from vipera_rs_b200.engine.planner import plan_memory, spec_cache_requests
+from vipera_rs_b200.parts.attention import GQAttention
 from vipera_rs_b200.parts.base import CacheBundle, FixedState, PagedKV
 from vipera_rs_b200.parts.rotary import QueryFactor
 
@@ -90,16 +91,21 @@ def test_tensor_names_of_a_written_folder():
 def test_what_layers_keep_between_steps():
     _, spec = spec_of("mixed")
     requests = spec_cache_requests(spec)
-    first = CacheBundle.of(left=PagedKV(2, 24, None, value_dim=16),
+    first = CacheBundle.of(left=PagedKV(2, 64, None),      # heads filled up to a tile
                            right=CacheBundle.of(conv=FixedState((3, 264)), scan=FixedState((6 * 24 * 20,))))
-    again = CacheBundle.of(left=PagedKV(3, 10, None, value_dim=14),
+    again = CacheBundle.of(left=PagedKV(3, 64, None),
                            right=CacheBundle.of(conv=FixedState((2, 36 + 80)), scan=FixedState((4 * 40 * 9,))))
-    assert requests[0] == first and requests[1] == requests[3] == requests[5] == PagedKV(2, 16, None, value_dim=24)
-    assert requests[2] == requests[4] == requests[6] == again and requests[7] == PagedKV(1, 12, None, value_dim=8)
+    assert requests[0] == first and requests[1] == requests[3] == requests[5] == PagedKV(2, 64, None)
+    assert requests[2] == requests[4] == requests[6] == again and requests[7] == PagedKV(1, 64, None)
     groups, states = plan_groups(requests)
-    assert sorted(len(group.slots) for group in groups) == [1, 1, 3, 3] and len(states) == 8
+    assert sorted(len(group.slots) for group in groups) == [1, 3, 4] and len(states) == 8
     assert spec_cache_requests(spec_of("odd")[1])[1].members[1][1] == CacheBundle.of(scan=FixedState((21,)))   # one tap keeps nothing
     assert plan_memory(spec, 256, 4, "bfloat16", device_bytes=10**9)["feasible"]
+    # up to 64 values, up to 128, and heads no tile holds
+    sizes = [GQAttention._stored_sizes({"head_dim": d, "value_dim": dv, "tile_heads": True})
+             for d, dv in ((64, 64), (5, 9), (65, 8), (40, 72), (128, 128), (160, 8))]
+    assert sizes == [(64, 64), (64, 64), (128, 128), (128, 128), (128, 128), (160, 8)]
+    assert GQAttention._stored_sizes({"head_dim": 40}) == (40, 40)
 
 
 @pytest.mark.parametrize("coef,every", [(0.7, 13), (0.5, 1), (0.3, 5000), (1.2, 3), (0.25, 7.5)])

@@ -82,7 +82,7 @@ def test_heads_on_their_way_to_the_cache(heads, kv_heads, d, dv, rot, style, dty
     angle = torch.arange(40, dtype=F)[:, None] * 30.0 ** (-torch.arange(half, dtype=F) / half)
     code = {"neox": ops.ROPE_NEOX, "interleaved": ops.ROPE_INTERLEAVED, "none": ops.ROPE_NONE}[style]
     limit = 2e-6 if dtype == torch.float32 else 5e-3
-    for with_norm, with_factor in ((True, True), (True, False), (False, True)):
+    for with_norm, with_factor, norm_size in ((True, True, None), (True, False, d - 1 if d > rot else d), (False, True, None)):
         k_pool = torch.full((9, page, kv_heads, d), float("nan"), dtype=dtype, device=DEV)
         v_pool = torch.full((9, page, kv_heads, dv), float("nan"), dtype=dtype, device=DEV)
         q_out = torch.full((tokens, heads * d), float("nan"), dtype=dtype, device=DEV)
@@ -90,12 +90,12 @@ def test_heads_on_their_way_to_the_cache(heads, kv_heads, d, dv, rot, style, dty
                       positions=position.to(DEV), cos=angle.cos().float().to(DEV), sin=angle.sin().float().to(DEV), style=code,
                       k_pool=k_pool, v_pool=v_pool, token_entry=entry.to(DEV), block_table=table.to(DEV), page_size=page,
                       write_cache=True, q_norm=wq.to(DEV) if with_norm else None, k_norm=wk.to(DEV) if with_norm else None,
-                      eps=eps, q_factor=factor.to(DEV) if with_factor else None)
+                      eps=eps, q_factor=factor.to(DEV) if with_factor else None, norm_size=norm_size)
 
         def head(rows, weight, t):
             rows = rows.double()
             if with_norm:
-                rows = rows / torch.sqrt((rows * rows).mean(-1, keepdim=True) + eps) * weight.double()
+                rows = rows / torch.sqrt((rows * rows).sum(-1, keepdim=True) / (norm_size or d) + eps) * weight.double()
             out = rows.clone()
             if style != "none":
                 c, s = angle[int(position[t])].cos(), angle[int(position[t])].sin()

@@ -179,7 +179,7 @@ _NAMES = ("q", "k", "v", "o")
 def _attention_part(config: ZugutarConfig, m: Dict[str, Any]) -> PartSpec:
     return PartSpec("gqa_attention", {
         "hidden_size": config.width, "num_heads": m["heads"], "num_kv_heads": m["kv_heads"], "head_dim": m["dim"],
-        "value_dim": m["vdim"], "qkv_bias": False, "window": None, "output_gate": True,
+        "value_dim": m["vdim"], "qkv_bias": False, "window": None, "output_gate": True, "tile_heads": True,
         "query_temperature": m["q_temp"], "max_positions": config.max_positions, "softmax_scale": m["scale"],
         "position": PartSpec("none", {}), "projection_names": _NAMES})
 
@@ -193,7 +193,7 @@ def _parallel_part(config: ZugutarConfig, m: Dict[str, Any]) -> PartSpec:
     softmax = PartSpec("gqa_attention", {
         "hidden_size": config.width, "num_heads": left["heads"], "num_kv_heads": left["kv_heads"], "head_dim": left["dim"],
         "value_dim": left["vdim"], "qkv_bias": False, "window": None, "head_norm": True, "norm_eps": config.eps, "sink": True,
-        "output_gate": "heads", "softmax_scale": left["scale"], "position": position, "projection_names": _NAMES})
+        "output_gate": "heads", "tile_heads": True, "softmax_scale": left["scale"], "position": position, "projection_names": _NAMES})
     recurrence = PartSpec("mamba2", {
         "hidden_size": config.width, "num_heads": right["heads"], "value_dim": right["vdim"], "state": right["state"],
         "groups": right["groups"], "taps": right["conv"], "norm_groups": right["norm_groups"], "norm_eps": config.eps})

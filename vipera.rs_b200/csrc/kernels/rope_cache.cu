@@ -346,6 +346,7 @@ struct HeadRowsParams {
   long long row_stride;
   void* q_out;              // [tokens, heads, head_dim]
   int num_tokens, num_heads, num_kv_heads, head_dim, value_dim, rot_dims, style;
+  int norm_size;            // values a norm's mean is over (the rest of a head is zeros)
   const float* q_norm;
   const float* k_norm;
   float eps;
@@ -401,7 +402,7 @@ head_rows_kernel(const HeadRowsParams p) {
     sum = fmaf(x[j], x[j], sum);
   }
   if (gain) {
-    const float inverse = 1.0f / sqrtf(warp_sum(sum) / static_cast<float>(size) + p.eps);
+    const float inverse = 1.0f / sqrtf(warp_sum(sum) / static_cast<float>(p.norm_size) + p.eps);
 #pragma unroll
     for (int j = 0; j < kPerLane; ++j) {
       const int e = lane + 32 * j;
@@ -489,7 +490,7 @@ head_rows_vector_kernel(const HeadRowsParams p) {
 #pragma unroll
       for (int j = 0; j < PIECES; ++j)
         sum += x[n][j].x * x[n][j].x + x[n][j].y * x[n][j].y + x[n][j].z * x[n][j].z + x[n][j].w * x[n][j].w;
-      const float inverse = 1.0f / sqrtf(warp_sum(sum) / static_cast<float>(size) + p.eps);
+      const float inverse = 1.0f / sqrtf(warp_sum(sum) / static_cast<float>(p.norm_size) + p.eps);
 #pragma unroll
       for (int j = 0; j < PIECES; ++j) {
         const int e = 4 * (lane + 32 * j);
@@ -574,7 +575,7 @@ VIPERA_API int vipera_head_rows(const HeadRowsParams* params, int dtype, void* s
   const HeadRowsParams& p = *params;
   if (p.num_tokens <= 0) return VIPERA_OK;
   if (p.head_dim <= 0 || p.head_dim > kHeadMost || p.value_dim <= 0 || p.value_dim > kHeadMost || p.num_heads <= 0 ||
-      p.num_kv_heads <= 0 || p.rot_dims < 0 || (p.rot_dims & 1) || p.rot_dims > p.head_dim)
+      p.num_kv_heads <= 0 || p.rot_dims < 0 || (p.rot_dims & 1) || p.rot_dims > p.head_dim || p.norm_size <= 0)
     return VIPERA_BAD_SHAPE;
   if (!p.qkv || !p.q_out || !p.positions) return VIPERA_BAD_ARGUMENT;
   if (p.style != ROPE_NONE && p.rot_dims > 0 && (!p.cos_table || !p.sin_table)) return VIPERA_BAD_ARGUMENT;

@@ -408,7 +408,7 @@ class _HeadRowsParams(ctypes.Structure):
     _fields_ = [
         ("qkv", _c_void), ("row_stride", ctypes.c_longlong), ("q_out", _c_void),
         ("num_tokens", _c_int), ("num_heads", _c_int), ("num_kv_heads", _c_int), ("head_dim", _c_int), ("value_dim", _c_int),
-        ("rot_dims", _c_int), ("style", _c_int), ("q_norm", _c_void), ("k_norm", _c_void), ("eps", _c_float),
+        ("rot_dims", _c_int), ("style", _c_int), ("norm_size", _c_int), ("q_norm", _c_void), ("k_norm", _c_void), ("eps", _c_float),
         ("q_factor", _c_void), ("positions", _c_void), ("cos_table", _c_void), ("sin_table", _c_void),
         ("k_pool", _c_void), ("v_pool", _c_void), ("token_entry", _c_void), ("block_table", _c_void),
         ("table_width", _c_int), ("page_size", _c_int), ("write_cache", _c_int),
@@ -420,10 +420,11 @@ def head_rows(qkv: torch.Tensor, q_out: torch.Tensor, *, num_heads: int, num_kv_
               sin: Optional[torch.Tensor], style: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
               token_entry: torch.Tensor, block_table: torch.Tensor, page_size: int, write_cache: bool,
               q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None, eps: float = 0.0,
-              q_factor: Optional[torch.Tensor] = None) -> None:
+              q_factor: Optional[torch.Tensor] = None, norm_size: Optional[int] = None) -> None:
     """Heads of a float32 product [tokens, >= (heads + kv_heads) * d + kv_heads * value_dim] on their way to q_out
     [tokens, heads * d] and the cache: an RMS norm per head (``q_norm``, ``k_norm`` float32 [d], shared by all
-    heads, or None), rotation of a head's first ``rot_dims`` values, queries times ``q_factor[position]``."""
+    heads, or None; the mean is over ``norm_size`` values, by default d: a head may be filled up with zeros),
+    rotation of a head's first ``rot_dims`` values, queries times ``q_factor[position]``."""
     fn = _function("rope_cache", "vipera_head_rows", [ctypes.POINTER(_HeadRowsParams), _c_int, _c_void])
     _check_struct("rope_cache", "vipera_head_rows_params_size", _HeadRowsParams)
     count = qkv.shape[0]
@@ -450,6 +451,7 @@ def head_rows(qkv: torch.Tensor, q_out: torch.Tensor, *, num_heads: int, num_kv_
     p.qkv, p.row_stride, p.q_out = _gpu(qkv, "qkv", torch.float32), int(qkv.stride(0)), _gpu(q_out, "q_out")
     p.num_tokens, p.num_heads, p.num_kv_heads = int(count), int(num_heads), int(num_kv_heads)
     p.head_dim, p.value_dim, p.rot_dims, p.style = int(head_dim), int(value_dim), int(rot_dims), int(style)
+    p.norm_size = int(norm_size or head_dim)
     p.q_norm, p.k_norm, p.eps = _opt(q_norm, "q_norm", torch.float32), _opt(k_norm, "k_norm", torch.float32), float(eps)
     p.q_factor, p.positions = _opt(q_factor, "q_factor", torch.float32), _gpu(positions, "positions", torch.int32)
     p.cos_table, p.sin_table = _opt(cos, "cos", torch.float32), _opt(sin, "sin", torch.float32)

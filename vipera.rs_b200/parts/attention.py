@@ -49,7 +49,9 @@ class GQAttention(Mixer):
     divided by its own root mean square and multiplied by a weight per value that all heads share,
     ``<q>.norm.weight`` and ``<k>.norm.weight`` [head_dim], before the rotation); ``query_temperature``
     (``{"coef", "every"}``, with ``max_positions``: the query at position p is multiplied by
-    ``1 + coef ln(floor((p + 1) / every) + 1)``); ``value_mix``:
+    ``1 + coef ln(floor((p + 1) / every) + 1)``); ``tile_heads`` (true: heads of up to 128 values are kept filled
+    up with zeros to the size the tensor-core kernels are built for, 64 or 128, keys and values alike: zero rows
+    of the projections and zero columns of the output matrix, which change no score and no output); ``value_mix``:
     ``"source"`` publishes the values of the step's tokens as projected, ``"blend"`` caches
     ``(1 - b) v + b v_source`` with ``b = <prefix>.vmix.weight`` (a single number) and ``v_source`` what
     the source layer published for the same token earlier in the step (both kinds hold the tensor;
@@ -67,6 +69,17 @@ class GQAttention(Mixer):
     @staticmethod
     def _names(params):
         return params.get("projection_names", ("q_proj", "k_proj", "v_proj", "o_proj"))
+
+    @staticmethod
+    def _stored_sizes(params):
+        """(key size, value size) of a head as it is projected, cached and attended."""
+        d = int(params["head_dim"])
+        dv = int(params.get("value_dim") or d)
+        if params.get("tile_heads", False):
+            for size in ops.TC_ATTENTION_HEAD_DIMS:
+                if max(d, dv) <= size:
+                    return size, size
+        return d, dv
 
     @classmethod
     def schema(cls, params, prefix):
@@ -109,8 +122,13 @@ class GQAttention(Mixer):
         self.hidden = int(params["hidden_size"])
         self.num_heads = int(params["num_heads"])
         self.num_kv_heads = int(params["num_kv_heads"])
-        self.head_dim = int(params["head_dim"])
-        self.value_dim = int(params.get("value_dim") or self.head_dim)
+        own_dim = int(params["head_dim"])
+        own_value = int(params.get("value_dim") or own_dim)
+        self.head_dim, self.value_dim = self._stored_sizes(params)
+        filled = (self.head_dim, self.value_dim) != (own_dim, own_value)
+        if filled and any(params.get(key) for key in ("values_from_keys", "row_norm", "talking_heads", "value_mix", "qkv_bias")):
+            raise UnsupportedError(f"{prefix}: heads filled up to a tile do not come with values that are the keys, a norm over "
+                                   "whole rows, mixed head weights, blended values or biases")
         self.window = params.get("window")
         self.keep_first = int(params.get("keep_first") or 0) if self.window else 0
         self.sink = bool(params.get("sink", False))
@@ -155,7 +173,7 @@ class GQAttention(Mixer):
             if self.window or self.chunk or self.sink or self.gated or self.value_mix:
                 raise UnsupportedError("attention: mixed head weights come with a plain causal mask only")
             self.talk = tensors[f"{prefix}.talk.weight"].to(device=device, dtype=torch.float32).contiguous()
-        self.q_norm = self.k_norm = None
+        self.q_norm = self.k_norm = self.norm_size = None
         if self.row_norm:
             self.q_norm = tensors[f"{prefix}.{qn}.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
             self.k_norm = tensors[f"{prefix}.{kn}.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
@@ -163,8 +181,10 @@ class GQAttention(Mixer):
             if self.row_norm or self.values_from_keys or self.value_mix:
                 raise UnsupportedError("attention: a norm per head does not come with a norm over whole rows, blended values "
                                        "or values that are the keys")
-            self.q_norm = tensors[f"{prefix}.{qn}.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
-            self.k_norm = tensors[f"{prefix}.{kn}.norm.weight"].to(device=device, dtype=torch.float32).contiguous()
+            self.norm_size = own_dim
+            self.q_norm, self.k_norm = (
+                torch.nn.functional.pad(tensors[f"{prefix}.{n}.norm.weight"].to(device=device, dtype=torch.float32),
+                                        (0, self.head_dim - own_dim)).contiguous() for n in (qn, kn))
         if self.q_factor is not None and (self.row_norm or self.values_from_keys or self.value_mix):
             raise UnsupportedError("attention: queries that grow with their position do not come with a norm over whole rows, "
                                    "blended values or values that are the keys")
@@ -175,18 +195,34 @@ class GQAttention(Mixer):
             raise UnsupportedError("attention: an output gate or blended values do not come with a norm over whole "
                                    "rows or values that are the keys")
         names = (qn, kn) if self.values_from_keys else (qn, kn, vn)
+
+        def rows_of(name, size, to):
+            """A matrix of heads of `size` rows, each head filled up with zero rows."""
+            weight = tensors[f"{prefix}.{name}.weight"]
+            if size == to:
+                return weight
+            heads = weight.view(-1, size, weight.shape[1])
+            return torch.nn.functional.pad(heads, (0, 0, 0, to - size)).reshape(-1, weight.shape[1])
+
+        rows = [rows_of(n, *sizes) for n, sizes in zip(names, ((own_dim, self.head_dim), (own_dim, self.head_dim),
+                                                               (own_value, self.value_dim)))]
         # the gate reads the mixer's input like q, k and v: its rows are the last of the one product
-        self.gate_offset = sum(tensors[f"{prefix}.{n}.weight"].shape[0] for n in names)
+        self.gate_offset = sum(r.shape[0] for r in rows)
         if self.gated:
-            names = names + (params.get("gate_name", "g"),)
-        fused = torch.cat([tensors[f"{prefix}.{n}.weight"] for n in names], dim=0)
+            gate = params.get("gate_name", "g")
+            rows.append(rows_of(gate, 1, 1) if self.gate_per_head else rows_of(gate, own_value, self.value_dim))
+        fused = torch.cat(rows, dim=0)
         bias = None
         if params.get("qkv_bias", False):
             bias = torch.cat([tensors[f"{prefix}.{n}.bias"].to(torch.float32) for n in (qn, kn, vn)], dim=0)
             if self.gated:
                 bias = torch.cat([bias, torch.zeros(fused.shape[0] - bias.shape[0])])
         self.qkv = Linear(fused, dtype, device, bias=bias)
-        self.out = Linear(tensors[f"{prefix}.{on}.weight"], dtype, device)
+        out_weight = tensors[f"{prefix}.{on}.weight"]
+        if own_value != self.value_dim:
+            out_weight = torch.nn.functional.pad(out_weight.view(self.hidden, self.num_heads, own_value),
+                                                 (0, self.value_dim - own_value)).reshape(self.hidden, -1)
+        self.out = Linear(out_weight, dtype, device)
         position = params["position"]
         self.position = POSITION_ENCODINGS.find(position.kind)(position.params, prefix, tensors, dtype, device)
         self.rot_dims = int(getattr(self.position, "rot_dims", self.head_dim))
@@ -224,17 +260,17 @@ class GQAttention(Mixer):
 
     @classmethod
     def cache_request_for(cls, params):
-        value_dim = int(params.get("value_dim") or params["head_dim"])
+        head_dim, value_dim = cls._stored_sizes(params)
         window = params.get("window")
-        return PagedKV(int(params["num_kv_heads"]), int(params["head_dim"]), window,
-                       value_dim=value_dim if value_dim != int(params["head_dim"]) else None,
+        return PagedKV(int(params["num_kv_heads"]), head_dim, window,
+                       value_dim=value_dim if value_dim != head_dim else None,
                        keep_first=int(params.get("keep_first") or 0) if window else 0)
 
     @classmethod
     def workspace_bytes(cls, params, tokens, element_bytes):
-        dv = params.get("value_dim") or params["head_dim"]
-        q_width = params["num_heads"] * params["head_dim"]
-        qkv_width = q_width + params["num_kv_heads"] * (params["head_dim"] + dv)
+        d, dv = cls._stored_sizes(params)
+        q_width = params["num_heads"] * d
+        qkv_width = q_width + params["num_kv_heads"] * (d + dv)
         if params.get("output_gate", False):
             qkv_width += params["num_heads"] * (1 if params["output_gate"] == "heads" else dv)
         if params.get("value_mix"):
@@ -315,7 +351,7 @@ class GQAttention(Mixer):
                           rot_dims=self.rot_dims if style != ops.ROPE_NONE else 0, positions=ctx.positions, cos=cos, sin=sin,
                           style=style, k_pool=cache.k, v_pool=cache.v, token_entry=ctx.token_entry, block_table=table,
                           page_size=cache.page_size, write_cache=writes_cache, q_norm=self.q_norm, k_norm=self.k_norm,
-                          eps=self.norm_eps, q_factor=None if self.q_factor is None else self.q_factor.table())
+                          eps=self.norm_eps, norm_size=self.norm_size, q_factor=None if self.q_factor is None else self.q_factor.table())
         elif self.gated or self.value_mix:
             publish = blend_with = None
             if self.value_mix == "source":
