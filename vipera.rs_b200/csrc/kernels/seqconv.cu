@@ -37,7 +37,7 @@ struct ConvParams {
 
 __device__ __forceinline__ float conv_finish(float sum, float current, const ConvParams& p, float bias) {
   sum += bias;
-  if (p.activation == CONV_ACT_SILU) sum = sum / (1.0f + expf(-sum));
+  if (p.activation == CONV_ACT_SILU) sum = __fdividef(sum, 1.0f + expf(-sum));   // (two units in the last place; 0 for the far negative)
   if (p.add_input) sum += current;
   return sum;
 }
@@ -127,11 +127,7 @@ __global__ void __launch_bounds__(kConvThreads) causal_conv_kernel(const ConvPar
     const int row = begin - (taps - 1) + k;
     inputs[k] = (k < kConvSegment + taps - 1 && row >= 0 && row < p.num_tokens) ? p.x[static_cast<size_t>(row) * p.x_stride + c] : 0.0f;
   }
-#pragma unroll
-  for (int i = 0; i < kConvSegment; ++i) {
-    const int t = begin + i;
-    if (t >= p.num_tokens) break;
-    if (t - p.entry_starts[p.token_entry[t]] < taps - 1) continue;
+  auto output = [&](int i) {
     float sum = 0.0f, current = 0.0f;
 #pragma unroll
     for (int j = 0; j < MAXT; ++j) {
@@ -140,8 +136,18 @@ __global__ void __launch_bounds__(kConvThreads) causal_conv_kernel(const ConvPar
         if (j == taps - 1) current = inputs[i + j];
       }
     }
-    conv_store<TO>(p, t, c, conv_finish(sum, current, p, bias));
+    conv_store<TO>(p, begin + i, c, conv_finish(sum, current, p, bias));
+  };
+  const int entry = p.token_entry[begin];
+  if (begin - p.entry_starts[entry] >= taps - 1 && begin + kConvSegment <= p.entry_starts[entry + 1]) {
+    // the whole segment lies within one entry, behind its first tokens
+#pragma unroll
+    for (int i = 0; i < kConvSegment; ++i) output(i);
+    return;
   }
+#pragma unroll
+  for (int i = 0; i < kConvSegment; ++i)
+    if (begin + i < p.num_tokens && begin + i - p.entry_starts[p.token_entry[begin + i]] >= taps - 1) output(i);
 }
 
 // single != 0 promises that every entry brings at most one token (no segment jobs are needed
